@@ -209,8 +209,7 @@ class DeviceCache:
         if free and self._states:
             index = torch.tensor(free, dtype=torch.long, device=self.device)
             for records in self._states:
-                if records.is_floating_point():
-                    records.index_fill_(1, index, value)
+                records.index_fill_(1, index, value if records.is_floating_point() else -(1 << 30))
 
     def poison_free_pages(self, value: float = float("nan")) -> None:
         """Overwrite every page that no request holds (a test aid: stale reads then show)."""

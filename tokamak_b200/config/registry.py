@@ -149,3 +149,6 @@ def _load_builtin() -> None:
         from ..models import pukinex
         register_architecture(Architecture(pukinex.ARCHITECTURE, pukinex.parse_config, pukinex.model_spec,
                                            reads_tensor_shapes=True))
+    if "Puresun" not in _ARCHITECTURES:
+        from ..models import puresun
+        register_architecture(Architecture(puresun.ARCHITECTURE, puresun.parse_config, puresun.model_spec))

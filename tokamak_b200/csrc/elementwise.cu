@@ -5,6 +5,7 @@
 // type.  RMSNorm statistics are 32-bit as in the reference
 // (src/tokamak/model/layers.py:28-33).
 #include "common.cuh"
+#include "stacked_input.cuh"
 #include "timeline.cuh"
 
 namespace tk {
@@ -34,6 +35,87 @@ __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __re
     return;
   }
   for (int h = threadIdx.x; h < hidden; h += blockDim.x) out[h] = to_f32<T>(row[h]) * scale;
+}
+
+// resid[t, :] = float(table[ids[t], :]) * scale + float(pairs[row, :]), where row is a hash of the request's
+// previous token and this one, (prev * mul_prev + cur * mul_cur) mod buckets, and `buckets` (the table's last row)
+// for a request's first token.  The previous token is the one before in the step or, for the first token of a
+// request's portion, the one that last[slot] holds from the step before; the block of that first token also moves
+// last[slot] on to the portion's last token, after it has read it, so no other block touches the entry.
+// keep: a second copy of the rows, or null.
+struct EmbedBigramParams {
+  const void* table; const void* pairs;
+  const int* ids; const int* positions; const int* tok_req; const int* req_q_start; const int* req_q_len;
+  const int* req_slot;
+  int* last;                // [max_slots]
+  float* resid; float* keep;
+  int n_tokens, n_reqs, max_slots, hidden, vocab, buckets;
+  long long mul_prev, mul_cur;
+  float scale;
+  int* err;
+};
+
+template <typename T>
+__global__ void embed_bigram_kernel(EmbedBigramParams p) {
+  __shared__ int s_id, s_row;
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x;
+  if (threadIdx.x == 0) {
+    int id = p.ids[t], row = -1;
+    const int pos = p.positions[t], r = p.tok_req[t];
+    if (id < 0 || id >= p.vocab) {
+      set_error(p.err, kErrTokenId, t, id, p.vocab);
+      id = -1;
+    }
+    if (pos < 0) {
+      set_error(p.err, kErrPosition, t, pos, 0);
+    } else if (r < 0 || r >= p.n_reqs) {
+      set_error(p.err, kErrRequest, t, r, p.n_reqs);
+    } else {
+      const int first = p.req_q_start[r], end = first + p.req_q_len[r], slot = p.req_slot[r];
+      if (slot < 0 || slot >= p.max_slots || first < 0 || t < first || t >= end || end > p.n_tokens) {
+        set_error(p.err, kErrRequest, t, r, slot);
+      } else {
+        int prev = 0;
+        if (pos > 0) prev = t > first ? p.ids[t - 1] : p.last[slot];
+        if (t == first) p.last[slot] = p.ids[end - 1];
+        if (pos == 0) {
+          row = p.buckets;
+        } else if (prev < 0 || prev >= p.vocab) {
+          set_error(p.err, kErrTokenId, t, prev, p.vocab);
+        } else if (id >= 0) {
+          const long long hash = ((long long)prev * p.mul_prev + (long long)id * p.mul_cur) % p.buckets;
+          row = (int)(hash < 0 ? hash + p.buckets : hash);
+        }
+      }
+    }
+    s_id = id; s_row = row;
+  }
+  __syncthreads();
+  const int id = s_id, row = s_row;
+  const bool ok = id >= 0 && row >= 0;
+  const T* a = (const T*)p.table + (size_t)(ok ? id : 0) * p.hidden;
+  const T* b = (const T*)p.pairs + (size_t)(ok ? row : 0) * p.hidden;
+  float* out = p.resid + (size_t)t * p.hidden;
+  float* copy = p.keep != nullptr ? p.keep + (size_t)t * p.hidden : nullptr;
+  if ((p.hidden & 3) == 0) {
+    for (int h = threadIdx.x * 4; h < p.hidden; h += blockDim.x * 4) {
+      float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (ok) {
+        const float4 x = ld4<T>(a + h), y = ld4<T>(b + h);
+        v = make_float4(x.x * p.scale + y.x, x.y * p.scale + y.y, x.z * p.scale + y.z, x.w * p.scale + y.w);
+      }
+      *reinterpret_cast<float4*>(out + h) = v;
+      if (copy != nullptr) *reinterpret_cast<float4*>(copy + h) = v;
+    }
+    return;
+  }
+  for (int h = threadIdx.x; h < p.hidden; h += blockDim.x) {
+    const float v = ok ? to_f32<T>(a[h]) * p.scale + to_f32<T>(b[h]) : 0.0f;
+    out[h] = v;
+    if (copy != nullptr) copy[h] = v;
+  }
 }
 
 // x = resid[r] (+ delta[r]);  resid[r] = x (when written back);
@@ -259,6 +341,23 @@ TK_API int tk_embed_gather(const void* table, int dtype, const int* ids, float* 
   TK_DISPATCH_DTYPE(dtype, T,
                     e = tk::launch(tk::embed_gather_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream,
                                        (const T*)table, ids, resid, hidden, vocab, scale, accumulate, err));
+  return (int)e;
+}
+
+TK_API int tk_embed_bigram(const void* table, const void* pairs, int dtype, const int* ids, const int* positions,
+                           const int* tok_req, const int* req_q_start, const int* req_q_len, const int* req_slot, int* last,
+                           float* resid, float* keep, int n_tokens, int n_reqs, int max_slots, int hidden, int vocab,
+                           int buckets, long long mul_prev, long long mul_cur, float scale, int* err, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (buckets < 1 || hidden < 1 || last == nullptr) return (int)cudaErrorInvalidValue;
+  tk::EmbedBigramParams p;
+  p.table = table; p.pairs = pairs; p.ids = ids; p.positions = positions; p.tok_req = tok_req;
+  p.req_q_start = req_q_start; p.req_q_len = req_q_len; p.req_slot = req_slot; p.last = last;
+  p.resid = resid; p.keep = keep; p.n_tokens = n_tokens; p.n_reqs = n_reqs; p.max_slots = max_slots; p.hidden = hidden;
+  p.vocab = vocab; p.buckets = buckets; p.mul_prev = mul_prev; p.mul_cur = mul_cur; p.scale = scale; p.err = err;
+  const int threads = hidden >= 2048 ? 256 : (hidden >= 512 ? 128 : 64);
+  cudaError_t e = cudaSuccess;
+  TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::embed_bigram_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, p));
   return (int)e;
 }
 

@@ -5,8 +5,9 @@
 // A token's cache row is  [ c (rank) | k_rot (rot) ]:
 //   c     = x_c * rsqrt(mean(x_c^2) + eps) * w_c        the latent, RMS-normed with a plain weight
 //   k_rot = the rotated key part that all heads share: neighbouring pairs (x[2i], x[2i+1]) of its
-//           first rot_pairs * 2 elements turn by the angle of the token's position (the table holds
-//           cos and sin, already multiplied by any magnitude factor); the rest passes unchanged
+//           first rot_pairs * 2 elements (or, half-split, the pairs (x[i], x[i + rot_pairs])) turn by the
+//           angle of the token's position (the table holds cos and sin, already multiplied by any
+//           magnitude factor); the rest passes unchanged
 // and the scores are taken in the latent space: with q_abs[h] = W_uk[h]^T q_nope[h] (a product of
 // its own, given here as float32 [heads, tokens, rank])
 //   q_lat[t, h] = [ q_abs[h, t] | rotated q_rot[t, h] ]      float32
@@ -43,9 +44,35 @@ struct LatentPrepareParams {
   const int* req_kv_len;
   int* err;
   int n_tokens, n_reqs, heads, rank, rot, rot_pairs;
+  int halves;                 // pairs of elements rot_pairs apart instead of neighbours
   int page_size, max_pages, num_pages;
   float eps;
 };
+
+// Turns the rotated part x[off .. off + rot): store(e, value) is called once for every element.
+template <typename T, typename Store>
+__device__ __forceinline__ void turn_part(const LatentPrepareParams& p, size_t off, const float2* tab, Store store) {
+  if (p.halves) {
+    for (int e = threadIdx.x; e < p.rot; e += blockDim.x) {
+      const float x = stacked_ld<T>(p.in, off + e);
+      if (tab == nullptr || e >= 2 * p.rot_pairs) { store(e, x); continue; }
+      const bool first = e < p.rot_pairs;
+      const float2 cs = tab[first ? e : e - p.rot_pairs];
+      const float y = stacked_ld<T>(p.in, off + (first ? e + p.rot_pairs : e - p.rot_pairs));
+      store(e, first ? x * cs.x - y * cs.y : x * cs.x + y * cs.y);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; 2 * i < p.rot; i += blockDim.x) {
+    const float u = stacked_ld<T>(p.in, off + 2 * i);
+    const bool pair = 2 * i + 1 < p.rot;
+    const float w = pair ? stacked_ld<T>(p.in, off + 2 * i + 1) : 0.0f;
+    float2 cs = make_float2(1.0f, 0.0f);
+    if (tab != nullptr && i < p.rot_pairs) cs = tab[i];
+    store(2 * i, u * cs.x - w * cs.y);
+    if (pair) store(2 * i + 1, w * cs.x + u * cs.y);
+  }
+}
 
 template <typename T>
 __global__ void latent_prepare_kernel(LatentPrepareParams p) {
@@ -64,15 +91,7 @@ __global__ void latent_prepare_kernel(LatentPrepareParams p) {
     const float* src = p.q_abs + ((size_t)h * p.n_tokens + t) * p.rank;
     for (int e = threadIdx.x; e < p.rank; e += blockDim.x) dst[e] = src[e];
     const size_t qo = row + p.q_off + (size_t)h * p.q_head_cols + p.q_rot_off;
-    for (int i = threadIdx.x; 2 * i < p.rot; i += blockDim.x) {
-      const float u = stacked_ld<T>(p.in, qo + 2 * i);
-      const bool pair = 2 * i + 1 < p.rot;
-      const float w = pair ? stacked_ld<T>(p.in, qo + 2 * i + 1) : 0.0f;
-      float2 cs = make_float2(1.0f, 0.0f);
-      if (tab != nullptr && i < p.rot_pairs) cs = tab[i];
-      dst[p.rank + 2 * i] = u * cs.x - w * cs.y;
-      if (pair) dst[p.rank + 2 * i + 1] = w * cs.x + u * cs.y;
-    }
+    turn_part<T>(p, qo, tab, [&](int e, float v) { dst[p.rank + e] = v; });
     return;
   }
 
@@ -121,15 +140,7 @@ __global__ void latent_prepare_kernel(LatentPrepareParams p) {
     dst[e] = from_f32<T>(stacked_ld<T>(p.in, row + p.kv_off + e) * rstd * p.kv_norm_w[e]);
   }
   const size_t ko = row + p.kv_off + p.rank;
-  for (int i = threadIdx.x; 2 * i < p.rot; i += blockDim.x) {
-    const float u = stacked_ld<T>(p.in, ko + 2 * i);
-    const bool pair = 2 * i + 1 < p.rot;
-    const float w = pair ? stacked_ld<T>(p.in, ko + 2 * i + 1) : 0.0f;
-    float2 cs = make_float2(1.0f, 0.0f);
-    if (tab != nullptr && i < p.rot_pairs) cs = tab[i];
-    dst[p.rank + 2 * i] = from_f32<T>(u * cs.x - w * cs.y);
-    if (pair) dst[p.rank + 2 * i + 1] = from_f32<T>(w * cs.x + u * cs.y);
-  }
+  turn_part<T>(p, ko, tab, [&](int e, float v) { dst[p.rank + e] = from_f32<T>(v); });
 }
 
 // y[t, h * dv + e] = x[h, t, e] * sigmoid(gate[t, g_off + h * dv + e])   (no gate: g_off < 0)
@@ -161,7 +172,7 @@ TK_API int tk_latent_prepare(const void* x, const float* parts, int n_parts, lon
                              float* q_lat, void* cache, const float* rope_table, const int* positions,
                              const int* tok_req, const int* req_slot, const int* block_table, const int* req_q_len,
                              const int* req_kv_len, int* err, int n_tokens, int n_reqs, int heads, int rank, int rot,
-                             int rot_pairs, int page_size, int max_pages, int num_pages, float eps, int dtype,
+                             int rot_pairs, int halves, int page_size, int max_pages, int num_pages, float eps, int dtype,
                              cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if ((x == nullptr) == (parts == nullptr) || rank < 1 || rot < 0 || 2 * rot_pairs > rot || heads < 0 || heads > 65534 ||
@@ -176,7 +187,7 @@ TK_API int tk_latent_prepare(const void* x, const float* parts, int n_parts, lon
   p.q_abs = q_abs; p.q_lat = q_lat; p.cache = cache; p.rope_table = (const float2*)rope_table;
   p.positions = positions; p.tok_req = tok_req; p.req_slot = req_slot; p.block_table = block_table;
   p.req_q_len = req_q_len; p.req_kv_len = req_kv_len; p.err = err;
-  p.n_tokens = n_tokens; p.n_reqs = n_reqs; p.heads = heads; p.rank = rank; p.rot = rot; p.rot_pairs = rot_pairs;
+  p.n_tokens = n_tokens; p.n_reqs = n_reqs; p.heads = heads; p.rank = rank; p.rot = rot; p.rot_pairs = rot_pairs; p.halves = halves;
   p.page_size = page_size; p.max_pages = max_pages; p.num_pages = num_pages; p.eps = eps;
   const int widest = rank > cq_rank ? rank : cq_rank;
   const int threads = widest >= 256 ? 256 : (widest >= 128 ? 128 : 64);

@@ -17,6 +17,10 @@ _P = c_void_p
 # name -> argument types (every function returns a cudaError_t as int unless noted)
 _SIGNATURES: dict[str, list] = {
     "tk_embed_gather": [_P, c_int, _P, _P, c_int, c_int, c_int, c_float, c_int, _P, _P],
+    "tk_embed_bigram": [_P, _P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
+                        c_longlong, c_longlong, c_float, _P, _P],
+    "tk_sum_rmsnorm": [_P] + 2 * [_P, c_int, c_int, c_longlong, _P, _P] + [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float,
+                                                                          c_int, _P],
     "tk_step_begin": [_P, c_int, c_int, _P, c_int, _P, c_longlong, _P, _P, _P, _P, _P, c_int, c_int, _P, _P],
     "tk_decode_begin": [_P, c_int, c_int, _P, c_int, _P, c_longlong, _P, c_int, c_int, _P, _P, _P, _P, _P],
     "tk_sample_slots": [_P, c_longlong, _P, _P, c_int, _P, c_int, c_int, _P, _P],
@@ -39,7 +43,7 @@ _SIGNATURES: dict[str, list] = {
                            _P, c_int, _P],
     "tk_latent_prepare": [_P, _P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                           _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P,
-                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P],
+                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P],
     "tk_attention_latent": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_longlong, c_longlong,
                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P],
     "tk_attention_latent_takes": [c_int, c_int],
@@ -81,13 +85,14 @@ _SIGNATURES: dict[str, list] = {
                        c_float, c_int, _P],
     "tk_moe_tile_rows": [],
     "tk_moe_pad_rows": [],
-    "tk_moe_route": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "tk_moe_route": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                     _P],
     "tk_moe_gather": [_P, c_longlong, _P, _P, c_int, c_int, c_int, _P],
     "tk_moe_combine_rows": [_P, _P, _P, _P, c_int, c_int, c_int, _P],
-    "tk_moe_ffn": [_P, c_longlong, c_int, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "tk_moe_ffn": [_P, c_longlong, c_int, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P],
     "tk_moe_combine": [_P, _P, _P, c_int, c_int, c_int, _P],
     "tk_moe_small_max_pairs": [],
-    "tk_moe_small": [_P, c_longlong, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "tk_moe_small": [_P, c_longlong, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
     "tk_qkv_pairs": [_P, _P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P,
                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                      c_float, c_int, _P],

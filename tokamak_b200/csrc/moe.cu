@@ -1,10 +1,12 @@
-// A mixture of gated feed-forward experts with a sigmoid router.
+// A mixture of feed-forward experts, gated or not, with a sigmoid or a softmax router.
 //
-//   s = sigmoid(W_r h)                       scores, float32
+//   s = sigmoid(W_r h), or s = W_r h for a softmax router         scores, float32
 //   c = s + correction                       choice scores
 //   the experts form equal groups of neighbours; a group's score is the sum of its two largest c; only
 //   experts of the `keep` best groups can be chosen; the `top` experts with the largest c are chosen
-//   out = sum over the chosen e of s_e * W_down,e (act(W_gate,e h) * (W_up,e h))
+//   g_e = s_e, or, for a softmax router, exp(s_e) / sum of exp(s) over the chosen experts only
+//   out = sum over the chosen e of g_e * W_down,e (act(W_gate,e h) * (W_up,e h))       gated experts
+//   out = sum over the chosen e of g_e * W_down,e act(W_up,e h)                        ungated ones
 //
 // Five kernels.  moe_route_kernel: a block per token forms the logits, and its first warp makes the choice
 // (ties go to the lower index).  moe_sort_kernel: one block counts the (token, choice) pairs of every expert, lays the
@@ -58,7 +60,7 @@ __global__ void __launch_bounds__(kMoeRouteWarps * 32)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
                  const float* __restrict__ correction, int* __restrict__ chosen,
                  float* __restrict__ weights, int n_tokens, int width, int experts, int n_groups,
-                 int keep, int top) {
+                 int keep, int top, int softmax) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
@@ -84,7 +86,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
     }
     acc = warp_sum(acc);
     if (lane == 0) {
-      s[e] = 1.0f / (1.0f + expf(-acc));
+      s[e] = softmax ? acc : 1.0f / (1.0f + expf(-acc));
       c[e] = s[e] + (correction != nullptr ? correction[e] : 0.0f);
     }
   }
@@ -131,6 +133,13 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
       c[bi] = -INFINITY;
     }
     __syncwarp();
+  }
+  if (softmax && lane == 0) {       // the chosen experts' scores become weights that sum to one
+    float* w = weights + (size_t)t * top;
+    float m = w[0], sum = 0.0f;
+    for (int k = 1; k < top; ++k) m = fmaxf(m, w[k]);
+    for (int k = 0; k < top; ++k) { const float x = expf(w[k] - m); w[k] = x; sum += x; }
+    for (int k = 0; k < top; ++k) w[k] = w[k] / sum;
   }
 }
 
@@ -194,13 +203,17 @@ struct MoeFfnParams {
   int a_div;                // row of pair i is i / a_div (top for the tokens' rows, 1 for rows per pair)
   const void* b0;           // [experts, n_out, k] activation type
   const void* b1;           // the same for the second product of a gated unit, or null
-  void* out;                // row of pair i: gated [pairs, n_out] activation type, else float32
+  void* out;                // row of pair i, [pairs, n_out]: the sums float32, an activation in the activation type
   const int* order; const int* tiles; const int* n_tiles;
   int n_out, k, act;
 };
 
-template <typename T, bool kGated>
+// What a product leaves: its sums in float32, act(sum) in the activation type, or act(gate) * up.
+enum MoeProduct : int { kMoeSums = 0, kMoeUnary = 1, kMoeGated = 2 };
+
+template <typename T, int kMode>
 __global__ void __launch_bounds__(256) moe_ffn_kernel(MoeFfnParams p) {
+  constexpr bool kGated = kMode == kMoeGated;
   __shared__ float As[kMoeTileRows][kMoeTileK + 1];
   __shared__ float Bs[kGated ? 2 : 1][kMoeTileCols][kMoeTileK + 1];
   __shared__ int rows[kMoeTileRows];
@@ -256,6 +269,7 @@ __global__ void __launch_bounds__(256) moe_ffn_kernel(MoeFfnParams p) {
       const int c = n0 + tx + 16 * i;
       if (c >= p.n_out) continue;
       if (kGated) ((T*)p.out)[(size_t)pair * p.n_out + c] = from_f32<T>(glu_act(acc[j][i], p.act) * acc1[j][i]);
+      else if (kMode == kMoeUnary) ((T*)p.out)[(size_t)pair * p.n_out + c] = from_f32<T>(unary_act(acc[j][i], p.act));
       else ((float*)p.out)[(size_t)pair * p.n_out + c] = acc[j][i];
     }
   }
@@ -326,7 +340,7 @@ struct MoeSmallParams {
   long long a_stride;
   int a_div;
   const __nv_bfloat16* b;       // [experts, n_out, k], or the stacked gate/up matrix
-  void* out;                    // gated: bfloat16 [pairs, n_out]; else float32 [pairs, n_out]
+  void* out;                    // [pairs, n_out]: the sums float32, an activation (gated or not) bfloat16
   const int* chosen;            // [pairs]
   int pairs, experts, n_out, k, act, block;
 };
@@ -347,9 +361,10 @@ __device__ __forceinline__ void small_wait() {
 // Rows n_begin + warp, + kMoeSmallWarps, ... < n_end of expert e for `count` <= R staged input rows.
 // A warp's work is the sequence of (row, stage) items; item i + kMoeSmallStages - 1 is asked for before
 // item i is worked through.  ring: this lane's first piece; pieces of a stage are 512 bytes apart.
-template <int R, bool kGated>
+template <int R, int kMode>
 __device__ __forceinline__ void moe_small_rows(const MoeSmallParams& p, const __nv_bfloat16* xs, uint4* ring,
                                                const int* mine, int count, int e, int n_begin, int n_end) {
+  constexpr bool kGated = kMode == kMoeGated;
   constexpr int kSweeps = kGated ? kMoeSmallPieces / 2 : kMoeSmallPieces;     // sweeps of the warp over k in a stage
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int per_row = (p.k + kSweeps * 256 - 1) / (kSweeps * 256);
@@ -423,6 +438,7 @@ __device__ __forceinline__ void moe_small_rows(const MoeSmallParams& p, const __
         if (lane == 0) {
           const size_t at = (size_t)mine[r] * p.n_out + n;
           if (kGated) ((__nv_bfloat16*)p.out)[at] = __float2bfloat16_rn(glu_act(s0, p.act) * s1);
+          else if (kMode == kMoeUnary) ((__nv_bfloat16*)p.out)[at] = __float2bfloat16_rn(unary_act(s0, p.act));
           else ((float*)p.out)[at] = s0;
         }
       }
@@ -433,7 +449,7 @@ __device__ __forceinline__ void moe_small_rows(const MoeSmallParams& p, const __
   asm volatile("cp.async.wait_group 0;\n" ::: "memory");
 }
 
-template <bool kGated>
+template <int kMode>
 __global__ void __launch_bounds__(kMoeSmallWarps * 32) moe_small_kernel(MoeSmallParams p) {
   extern __shared__ __align__(16) unsigned char small_smem[];      // the warps' rings, then the staged input rows
   __shared__ unsigned live_bits[kMoeMaxExperts / 32];
@@ -499,8 +515,8 @@ __global__ void __launch_bounds__(kMoeSmallWarps * 32) moe_small_kernel(MoeSmall
             reinterpret_cast<const uint4*>(p.a + (size_t)(mine[first + r] / p.a_div) * p.a_stride)[c];
       }
       __syncthreads();
-      if (count <= 2) moe_small_rows<2, kGated>(p, xs, ring, mine + first, count, e, n_begin, n_end);
-      else moe_small_rows<4, kGated>(p, xs, ring, mine + first, count, e, n_begin, n_end);
+      if (count <= 2) moe_small_rows<2, kMode>(p, xs, ring, mine + first, count, e, n_begin, n_end);
+      else moe_small_rows<4, kMode>(p, xs, ring, mine + first, count, e, n_begin, n_end);
       __syncthreads();
     }
     g += n_end - n_begin;
@@ -515,7 +531,7 @@ TK_API int tk_moe_pad_rows() { return tk::kMoePadRows; }
 
 TK_API int tk_moe_route(const void* h, const float* router, const float* correction, int* chosen, float* weights,
                         int* order, int* tiles, int* n_tiles, int* pair_row, int* tile_expert, int max_pad_tiles,
-                        int n_tokens, int width, int experts, int n_groups, int keep, int top, int dtype,
+                        int n_tokens, int width, int experts, int n_groups, int keep, int top, int softmax, int dtype,
                         cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (experts < 1 || experts > tk::kMoeMaxExperts || n_groups < 1 || experts % n_groups || keep < 1 || keep > n_groups ||
@@ -526,7 +542,7 @@ TK_API int tk_moe_route(const void* h, const float* router, const float* correct
   cudaError_t e = cudaSuccess;
   TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::moe_route_kernel<T>, dim3((unsigned)n_tokens),
                                              dim3(tk::kMoeRouteWarps * 32), smem, stream, (const T*)h, router, correction, chosen,
-                                             weights, n_tokens, width, experts, n_groups, keep, top));
+                                             weights, n_tokens, width, experts, n_groups, keep, top, softmax));
   if (e != cudaSuccess) return (int)e;
   e = tk::launch(tk::moe_sort_kernel, dim3(1), dim3(1024), 0, stream, (const int*)chosen, order, tiles, n_tiles,
                  n_tokens * top, experts, pair_row, tile_expert, max_pad_tiles);
@@ -553,23 +569,25 @@ TK_API int tk_moe_combine_rows(const void* y, const float* weights, const int* p
                          (const __nv_bfloat16*)y, weights, pair_row, out, n_tokens, width, top);
 }
 
-// gated != 0: out[pair] = act(a[pair / a_div] b0^T) * (a[pair / a_div] b1^T) in the activation type;
-// else out[pair] = a[pair / a_div] b0^T in float32.
+// mode kMoeGated: out[pair] = act(a[pair / a_div] b0^T) * (a[pair / a_div] b1^T) in the activation type;
+// kMoeUnary: out[pair] = act(a[pair / a_div] b0^T) in the activation type; kMoeSums: a[pair / a_div] b0^T in float32.
 TK_API int tk_moe_ffn(const void* a, long long a_stride, int a_div, const void* b0, const void* b1, void* out,
                       const int* order, const int* tiles, const int* n_tiles, int max_tiles, int n_out, int k, int act,
-                      int dtype, cudaStream_t stream) {
+                      int mode, int dtype, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
-  if (n_out < 1 || k < 1 || a_div < 1) return (int)cudaErrorInvalidValue;
+  if (n_out < 1 || k < 1 || a_div < 1 || (mode == tk::kMoeGated) != (b1 != nullptr)) return (int)cudaErrorInvalidValue;
   tk::MoeFfnParams p;
   p.a = a; p.a_stride = a_stride; p.a_div = a_div; p.b0 = b0; p.b1 = b1; p.out = out;
   p.order = order; p.tiles = tiles; p.n_tiles = n_tiles; p.n_out = n_out; p.k = k; p.act = act;
   const dim3 grid((unsigned)max_tiles, (unsigned)((n_out + tk::kMoeTileCols - 1) / tk::kMoeTileCols));
   cudaError_t e = cudaSuccess;
-  if (b1 != nullptr) {
-    TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::moe_ffn_kernel<T, true>, grid, dim3(256), 0, stream, p));
-  } else {
-    TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::moe_ffn_kernel<T, false>, grid, dim3(256), 0, stream, p));
-  }
+#define TK_MOE_FFN(M) \
+  TK_DISPATCH_DTYPE(dtype, T, (e = tk::launch(tk::moe_ffn_kernel<T, M>, grid, dim3(256), 0, stream, p)))
+  if (mode == tk::kMoeGated) { TK_MOE_FFN(tk::kMoeGated); }
+  else if (mode == tk::kMoeUnary) { TK_MOE_FFN(tk::kMoeUnary); }
+  else if (mode == tk::kMoeSums) { TK_MOE_FFN(tk::kMoeSums); }
+  else return (int)cudaErrorInvalidValue;
+#undef TK_MOE_FFN
   return (int)e;
 }
 
@@ -583,14 +601,15 @@ TK_API int tk_moe_combine(const float* y, const float* weights, float* out, int 
 
 TK_API int tk_moe_small_max_pairs() { return tk::kMoeSmallMaxPairs; }
 
-// bfloat16.  block > 0: b is the stacked gate/up matrix [experts, 2 n_out, k] (alternating blocks of `block`
-// rows), out[pair] = act(gate) * up in bfloat16; block == 0: b is [experts, n_out, k], out[pair] float32.
+// bfloat16.  kMoeGated: b is the stacked gate/up matrix [experts, 2 n_out, k] (alternating blocks of `block`
+// rows), out[pair] = act(gate) * up in bfloat16; kMoeUnary: b is [experts, n_out, k], out[pair] = act(sum) in
+// bfloat16; kMoeSums: the same b, out[pair] float32.
 TK_API int tk_moe_small(const void* a, long long a_stride, int a_div, const void* b, void* out, const int* chosen,
-                        int pairs, int experts, int n_out, int k, int act, int block, cudaStream_t stream) {
+                        int pairs, int experts, int n_out, int k, int act, int block, int mode, cudaStream_t stream) {
   if (pairs <= 0) return 0;
   const size_t smem = (size_t)tk::kMoeSmallRing + (size_t)tk::kMoeSmallRows * k * sizeof(__nv_bfloat16);
   if (pairs > tk::kMoeSmallMaxPairs || experts < 1 || experts > tk::kMoeMaxExperts || n_out < 1 || k < 8 || k % 8 ||
-      a_stride % 8 || a_div < 1 || block < 0 || (block > 0 && n_out % block) || smem > 200 * 1024 ||
+      a_stride % 8 || a_div < 1 || (mode == tk::kMoeGated && (block < 1 || n_out % block)) || smem > 200 * 1024 ||
       ((uintptr_t)a & 15u) || ((uintptr_t)b & 15u)) {
     return (int)cudaErrorInvalidValue;
   }
@@ -616,7 +635,10 @@ TK_API int tk_moe_small(const void* a, long long a_stride, int a_div, const void
     const long long blocks = (long long)sms * per_sm < most ? (long long)sms * per_sm : most;                           \
     e = tk::launch(tk::moe_small_kernel<G>, dim3((unsigned)blocks), dim3(tk::kMoeSmallWarps * 32), smem, stream, p);    \
   } while (0)
-  if (block > 0) { TK_MOE_SMALL(true); } else { TK_MOE_SMALL(false); }
+  if (mode == tk::kMoeGated) { TK_MOE_SMALL(tk::kMoeGated); }
+  else if (mode == tk::kMoeUnary) { TK_MOE_SMALL(tk::kMoeUnary); }
+  else if (mode == tk::kMoeSums) { TK_MOE_SMALL(tk::kMoeSums); }
+  else return (int)cudaErrorInvalidValue;
 #undef TK_MOE_SMALL
   return (int)e;
 }

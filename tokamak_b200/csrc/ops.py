@@ -87,6 +87,33 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, resid: torch.Tensor, er
            "embed_gather")
 
 
+def embed_bigram(table: torch.Tensor, pairs: torch.Tensor, last: torch.Tensor, step, resid: torch.Tensor, *,
+                 mul_prev: int, mul_cur: int, scale: float = 1.0, keep: torch.Tensor | None = None) -> None:
+    """``resid[t] = float32(table[id_t]) * scale + float32(pairs[row_t])`` with ``row_t = (id_(t-1) mul_prev + id_t
+    mul_cur) mod B`` for the token before in the same request, ``B`` (the last row of ``pairs`` ``[B + 1, hidden]``)
+    for a request's first token.  ``last`` (int32 ``[slots, 1]``) holds every request's last token between steps and
+    is moved on.  ``keep``: a second float32 copy of the rows."""
+    _want(table, None, "table"); _want(pairs, table.dtype, "pairs"); _want(last, torch.int32, "last")
+    _want(resid, torch.float32, "resid")
+    n = step.token_ids.numel()
+    vocab, hidden = table.shape
+    buckets = pairs.shape[0] - 1
+    if pairs.shape[1] != hidden or buckets < 1 or resid.shape[-1] != hidden or resid.numel() < n * hidden:
+        raise KernelError("the tables and the rows do not fit")
+    if keep is not None:
+        _want(keep, torch.float32, "keep")
+        if keep.shape != resid.shape:
+            raise KernelError("keep must have the shape of resid")
+    for name in ("token_ids", "positions", "tok_req", "req_q_start", "req_q_len", "req_slot"):
+        _want(getattr(step, name), torch.int32, name)
+    _check(_lib().tk_embed_bigram(table.data_ptr(), pairs.data_ptr(), dtype_code(table.dtype), step.token_ids.data_ptr(),
+                                     step.positions.data_ptr(), step.tok_req.data_ptr(), step.req_q_start.data_ptr(),
+                                     step.req_q_len.data_ptr(), step.req_slot.data_ptr(), last.data_ptr(),
+                                     resid.data_ptr(), _ptr(keep), n, step.req_slot.numel(), last.shape[0], hidden, vocab,
+                                     buckets, int(mul_prev), int(mul_cur), float(scale), step.err.data_ptr(), _stream()),
+           "embed_bigram")
+
+
 class UpdateBuffers:
     """Device side of the update list that the kernels opening a step apply (``step_state.cu``):
     the list itself, the engine's slot records and the flat block tables it writes into."""
@@ -236,6 +263,52 @@ def add_rmsnorm(resid: torch.Tensor, delta: torch.Tensor | None, weight: torch.T
     _check(_lib().tk_add_rmsnorm(resid.data_ptr(), _ptr(delta), _ptr(parts), n_parts, part_stride,
                                     weight.data_ptr(), out.data_ptr(), _ptr(rows), n_rows, hidden,
                                     float(eps), dtype_code(out.dtype), _stream()), "add_rmsnorm")
+
+
+SUM_NORM_TERMS = 2      # branches that one call of sum_rmsnorm adds
+
+
+def sum_rmsnorm(resid: torch.Tensor, terms, out: torch.Tensor, weight: torch.Tensor, eps: float, *,
+                rows: torch.Tensor | None = None, extra: torch.Tensor | None = None,
+                vector: torch.Tensor | None = None) -> None:
+    """``x = resid + terms[0] + terms[1] + extra + vector`` in float32 (written back unless ``rows`` selects rows), then
+    ``out = weight * x * rsqrt(mean x^2 + eps)``.  A term (at most ``SUM_NORM_TERMS``) is a branch's output in the
+    activation type, the float32 partial sums of a split product or :class:`WeightedRows`; ``extra`` is float32 rows
+    like ``resid``, ``vector`` one float32 row that every token receives."""
+    _want(resid, torch.float32, "resid"); _want(weight, torch.float32, "weight"); _want(out, None, "out")
+    n, width = resid.shape
+    if len(terms) > SUM_NORM_TERMS:
+        raise KernelError(f"at most {SUM_NORM_TERMS} branches join at a time")
+    if weight.numel() != width or out.shape[-1] != width:
+        raise KernelError("norm width mismatch")
+    args = []
+    for term in terms:
+        if tuple(term.shape[-2:]) != (n, width):
+            raise KernelError("a branch and the stream differ in shape")
+        if isinstance(term, WeightedRows):
+            _want(term.y, None, "y"); _want(term.weights, torch.float32, "weights")
+            args += [term.y.data_ptr(), 3 if term.y.dtype == torch.bfloat16 else 4, term.weights.shape[1], 0,
+                     term.weights.data_ptr(), _ptr(term.pair_row)]
+        elif term.dim() == 3:
+            _want(term, torch.float32, "partial sums")
+            args += [term.data_ptr(), 2, term.shape[0], term.stride(0), None, None]
+        else:
+            _want(term, out.dtype, "branch")
+            args += [term.data_ptr(), 1, 1, 0, None, None]
+    args += [None, 0, 0, 0, None, None] * (SUM_NORM_TERMS - len(terms))
+    for name, t, shape in (("extra", extra, (n, width)), ("vector", vector, (width,))):
+        if t is not None:
+            _want(t, torch.float32, name)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"{name} must be {shape}")
+    if rows is not None:
+        _want(rows, torch.int32, "rows")
+    n_rows = rows.numel() if rows is not None else n
+    if out.numel() < n_rows * width:
+        raise KernelError("out is too small")
+    _check(_lib().tk_sum_rmsnorm(resid.data_ptr(), *args, _ptr(extra), _ptr(vector), weight.data_ptr(), out.data_ptr(),
+                                    _ptr(rows), n_rows, n, width, float(eps), dtype_code(out.dtype), _stream()),
+           "sum_rmsnorm")
 
 
 GLU_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
@@ -1024,10 +1097,16 @@ def moe_pad_rows() -> int:
     return _lib().tk_moe_pad_rows()
 
 
-def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, *, top: int, n_groups: int,
-              keep: int, padded: bool = False) -> MoeRouting:
-    """Scores ``sigmoid(h router^T)`` in float32, choice by score plus ``correction`` among the ``keep`` groups
-    of neighbouring experts whose two best choice scores add up highest, weights the plain scores."""
+ROUTER_KINDS = {"sigmoid": 0, "softmax": 1}
+
+
+def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, *, top: int, n_groups: int = 1,
+              keep: int = 1, padded: bool = False, kind: str = "sigmoid") -> MoeRouting:
+    """Scores ``sigmoid(h router^T)`` in float32 (``kind="softmax"``: the logits themselves), choice by score plus
+    ``correction`` among the ``keep`` groups of neighbouring experts whose two best choice scores add up highest,
+    weights the plain scores (``softmax``: their softmax over the chosen experts only)."""
+    if kind not in ROUTER_KINDS:
+        raise KernelError(f"unknown router {kind!r}; known: {', '.join(ROUTER_KINDS)}")
     _want(h, None, "h"); _want(router, torch.float32, "router")
     n, width = h.shape
     experts = router.shape[0]
@@ -1050,14 +1129,52 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
     _check(_lib().tk_moe_route(h.data_ptr(), router.data_ptr(), _ptr(correction), chosen.data_ptr(), weights.data_ptr(),
                                   order.data_ptr(), tiles.data_ptr(), n_tiles.data_ptr(), _ptr(pair_row), _ptr(tile_expert),
                                   tile_expert.numel() if padded else 0, n, width, experts, n_groups,
-                                  keep, top, dtype_code(h.dtype), _stream()), "moe_route")
+                                  keep, top, ROUTER_KINDS[kind], dtype_code(h.dtype), _stream()), "moe_route")
     return MoeRouting(chosen, weights, order, tiles, n_tiles, max_tiles, pair_row, tile_expert)
 
 
-def moe_tc_takes(dtype: torch.dtype, width: int, ff: int) -> bool:
+MOE_SUMS, MOE_UNARY, MOE_GATED = 0, 1, 2        # what a product of the experts leaves (csrc/moe.cu)
+
+
+@dataclass
+class WeightedRows:
+    """The experts' outputs of a step before their weighted sum: token ``t``'s is the float32 sum over its
+    choices ``k`` of ``weights[t, k] * y[row(t, k)]``, with ``row`` the entry of ``pair_row`` or, without one, ``t *
+    top + k``.  A kernel that reads it forms the sum itself (:func:`sum_rmsnorm`); :meth:`combine` is the sum."""
+
+    y: torch.Tensor                     # [rows, width] bfloat16 or float32
+    weights: torch.Tensor               # [tokens, top] float32
+    pair_row: torch.Tensor | None       # [tokens * top] int32
+
+    @property
+    def shape(self) -> tuple[int, int]:
+        return self.weights.shape[0], self.y.shape[1]
+
+    def combine(self) -> torch.Tensor:
+        n, width = self.shape
+        top = self.weights.shape[1]
+        out = torch.empty((n, width), dtype=torch.float32, device=self.y.device)
+        if self.y.dtype == torch.bfloat16:
+            _check(_lib().tk_moe_combine_rows(self.y.data_ptr(), self.weights.data_ptr(), self.pair_row.data_ptr(),
+                                              out.data_ptr(), n, width, top, _stream()), "moe_combine_rows")
+        else:
+            _check(_lib().tk_moe_combine(self.y.data_ptr(), self.weights.data_ptr(), out.data_ptr(), n, width, top,
+                                         _stream()), "moe_combine")
+        return out
+
+
+def _moe_activation(activation: str, gated: bool) -> int:
+    known = GLU_ACTIVATIONS if gated else UNARY_ACTIVATIONS
+    if activation not in known:
+        raise KernelError(f"unknown activation {activation!r}")
+    return known[activation]
+
+
+def moe_tc_takes(dtype: torch.dtype, width: int, ff: int, gated: bool = True) -> bool:
     """Whether :func:`moe_experts_tc` runs these sizes: bfloat16, an inner size in whole blocks of the fused
-    activation, rows that TMA and 16-byte stores can address."""
-    return dtype == torch.bfloat16 and ff % SWIGLU_TILE_BLOCK == 0 and width % 8 == 0 and PAIR_GEMM_POLICY != "off"
+    gated activation, rows that TMA and 16-byte stores can address."""
+    return (dtype == torch.bfloat16 and ff % (SWIGLU_TILE_BLOCK if gated else 8) == 0 and width % 8 == 0
+            and PAIR_GEMM_POLICY != "off")
 
 
 def moe_stack_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
@@ -1069,107 +1186,110 @@ def moe_stack_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
                        dim=2).reshape(experts, 2 * ff, width).contiguous()
 
 
-def moe_experts_tc(h: torch.Tensor, routing: MoeRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, err: torch.Tensor,
-                   activation: str = "silu") -> torch.Tensor:
-    """:func:`moe_experts` on the tensor cores (bfloat16): the tokens' rows are copied into the padded layout
-    of ``routing``, the grouped product on pairs of SMs forms ``act(gate) * up`` in its epilogue and then the
-    down product, row for row, and the weighted sum reads the pairs' rows.  ``w_gate_up`` is what
-    :func:`moe_stack_gate_up` returns, ``w_down`` ``[experts, width, ff]``.  float32 ``[tokens, width]``."""
-    _want(h, torch.bfloat16, "h"); _want(w_gate_up, torch.bfloat16, "w_gate_up"); _want(w_down, torch.bfloat16, "w_down")
+def _moe_sizes(h: torch.Tensor, w_first: torch.Tensor, w_down: torch.Tensor, gated: bool, what: str) -> tuple:
+    """``(tokens, width, experts, ff)`` of a step through ``w_first`` (stacked gate/up, or up alone) and ``w_down``."""
+    _want(h, torch.bfloat16, "h"); _want(w_first, torch.bfloat16, "w_first"); _want(w_down, torch.bfloat16, "w_down")
     n, width = h.shape
-    experts, ff2, _ = w_gate_up.shape
-    ff = ff2 // 2
+    experts, _, ff = w_down.shape
+    if w_first.shape != (experts, (2 if gated else 1) * ff, width) or w_down.shape != (experts, width, ff):
+        raise KernelError(f"{what}: the weights must be stacked for these sizes")
+    return n, width, experts, ff
+
+
+def moe_experts_tc(h: torch.Tensor, routing: MoeRouting, w_first: torch.Tensor, w_down: torch.Tensor, err: torch.Tensor,
+                   activation: str = "silu", gated: bool = True, combine: bool = True):
+    """:func:`moe_experts` on the tensor cores (bfloat16): the tokens' rows are copied into the padded layout
+    of ``routing``, the grouped product on pairs of SMs forms ``act(gate) * up`` (or ``act(up)``) in its epilogue
+    and then the down product, row for row, and the weighted sum reads the pairs' rows.  ``w_first`` is what
+    :func:`moe_stack_gate_up` returns or, with ``gated=False``, ``[experts, ff, width]``; ``w_down`` is ``[experts,
+    width, ff]``.  float32 ``[tokens, width]``, or :class:`WeightedRows` with ``combine=False``."""
+    n, width, experts, ff = _moe_sizes(h, w_first, w_down, gated, "moe_experts_tc")
     top = routing.chosen.shape[1]
-    if routing.pair_row is None or w_gate_up.shape != (experts, 2 * ff, width) or w_down.shape != (experts, width, ff):
-        raise KernelError("moe_experts_tc: the routing must be padded and the weights stacked for these sizes")
-    if not moe_tc_takes(h.dtype, width, ff) or h.stride(1) != 1 or h.stride(0) % 8:
+    if routing.pair_row is None:
+        raise KernelError("moe_experts_tc: the routing must be padded")
+    if not moe_tc_takes(h.dtype, width, ff, gated) or h.stride(1) != 1 or h.stride(0) % 8:
         raise KernelError("moe_experts_tc does not take these sizes")
-    if activation not in GLU_ACTIVATIONS:
-        raise KernelError(f"unknown activation {activation!r}")
+    act_code = _moe_activation(activation, gated)
     flush_chains()
     lib, r = _lib(), routing
     rows = r.tile_expert.numel() * moe_pad_rows()
     xs = torch.empty((rows, width), dtype=torch.bfloat16, device=h.device)
     act = torch.empty((rows, ff), dtype=torch.bfloat16, device=h.device)
     y = torch.empty((rows, width), dtype=torch.bfloat16, device=h.device)
-    out = torch.empty((n, width), dtype=torch.float32, device=h.device)
     _check(lib.tk_moe_gather(h.data_ptr(), h.stride(0), xs.data_ptr(), r.pair_row.data_ptr(), n, top, width, _stream()),
            "moe_gather")
-    _check(lib.tk_gemm_bf16_pair_grouped(xs.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), err.data_ptr(),
-                                         r.tile_expert.data_ptr(), rows, experts, 2 * ff, width, width, width, ff,
-                                         1 + GLU_ACTIVATIONS[activation], _stream()), "gemm_pair_grouped (gate, up)")
+    _check(lib.tk_gemm_bf16_pair_grouped(xs.data_ptr(), w_first.data_ptr(), act.data_ptr(), err.data_ptr(),
+                                         r.tile_expert.data_ptr(), rows, experts, (2 if gated else 1) * ff, width, width,
+                                         width, ff, (1 if gated else 3) + act_code, _stream()),
+           "gemm_pair_grouped (first product)")
     _check(lib.tk_gemm_bf16_pair_grouped(act.data_ptr(), w_down.data_ptr(), y.data_ptr(), err.data_ptr(),
                                          r.tile_expert.data_ptr(), rows, experts, width, ff, ff, ff, width, 0, _stream()),
            "gemm_pair_grouped (down)")
-    _check(lib.tk_moe_combine_rows(y.data_ptr(), r.weights.data_ptr(), r.pair_row.data_ptr(), out.data_ptr(), n, width,
-                                   top, _stream()), "moe_combine_rows")
-    return out
+    out = WeightedRows(y, r.weights, r.pair_row)
+    return out.combine() if combine else out
 
 
-def moe_small_takes(n_tokens: int, top: int, width: int, ff: int) -> bool:
+def moe_small_takes(n_tokens: int, top: int, width: int, ff: int, gated: bool = True) -> bool:
     """Whether :func:`moe_experts_small` runs a step of these sizes: few enough (token, choice) pairs that an
     expert's weights are better streamed once past them than multiplied in whole tiles."""
-    return (n_tokens * top <= MOE_SMALL_PAIRS and width % 8 == 0 and ff % 8 == 0 and ff % SWIGLU_TILE_BLOCK == 0
+    return (n_tokens * top <= MOE_SMALL_PAIRS and width % 8 == 0 and ff % (SWIGLU_TILE_BLOCK if gated else 8) == 0
             and 65536 + 8 * max(width, ff) <= 200 * 1024)
 
 
-def moe_experts_small(h: torch.Tensor, routing: MoeRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                      activation: str = "silu") -> torch.Tensor:
+def moe_experts_small(h: torch.Tensor, routing: MoeRouting, w_first: torch.Tensor, w_down: torch.Tensor,
+                      activation: str = "silu", gated: bool = True, combine: bool = True):
     """:func:`moe_experts` for steps of few tokens (bfloat16): only the experts that some token chose are
     read, once, a warp an output row; the sums are float32, the rows between the two products bfloat16.
-    ``w_gate_up`` is what :func:`moe_stack_gate_up` returns.  float32 ``[tokens, width]``."""
-    _want(h, torch.bfloat16, "h"); _want(w_gate_up, torch.bfloat16, "w_gate_up"); _want(w_down, torch.bfloat16, "w_down")
-    n, width = h.shape
-    experts, ff2, _ = w_gate_up.shape
-    ff = ff2 // 2
+    ``w_first`` and the result as in :func:`moe_experts_tc`."""
+    n, width, experts, ff = _moe_sizes(h, w_first, w_down, gated, "moe_experts_small")
     top = routing.chosen.shape[1]
-    if w_gate_up.shape != (experts, 2 * ff, width) or w_down.shape != (experts, width, ff):
-        raise KernelError("moe_experts_small: the weights must be stacked for these sizes")
-    if not moe_small_takes(n, top, width, ff) or h.stride(1) != 1 or h.stride(0) % 8:
+    if not moe_small_takes(n, top, width, ff, gated) or h.stride(1) != 1 or h.stride(0) % 8:
         raise KernelError("moe_experts_small does not take these sizes")
-    if activation not in GLU_ACTIVATIONS:
-        raise KernelError(f"unknown activation {activation!r}")
+    act_code = _moe_activation(activation, gated)
     flush_chains()
     lib, pairs = _lib(), n * top
     act = torch.empty((pairs, ff), dtype=torch.bfloat16, device=h.device)
     y = torch.empty((pairs, width), dtype=torch.float32, device=h.device)
-    out = torch.empty((n, width), dtype=torch.float32, device=h.device)
-    _check(lib.tk_moe_small(h.data_ptr(), h.stride(0), top, w_gate_up.data_ptr(), act.data_ptr(),
-                            routing.chosen.data_ptr(), pairs, experts, ff, width, GLU_ACTIVATIONS[activation],
-                            SWIGLU_TILE_BLOCK, _stream()), "moe_small (gate, up)")
+    _check(lib.tk_moe_small(h.data_ptr(), h.stride(0), top, w_first.data_ptr(), act.data_ptr(),
+                            routing.chosen.data_ptr(), pairs, experts, ff, width, act_code, SWIGLU_TILE_BLOCK,
+                            MOE_GATED if gated else MOE_UNARY, _stream()), "moe_small (first product)")
     _check(lib.tk_moe_small(act.data_ptr(), ff, 1, w_down.data_ptr(), y.data_ptr(), routing.chosen.data_ptr(), pairs,
-                            experts, width, ff, 0, 0, _stream()), "moe_small (down)")
-    _check(lib.tk_moe_combine(y.data_ptr(), routing.weights.data_ptr(), out.data_ptr(), n, width, top, _stream()),
-           "moe_combine")
-    return out
+                            experts, width, ff, 0, 0, MOE_SUMS, _stream()), "moe_small (down)")
+    out = WeightedRows(y, routing.weights, None)
+    return out.combine() if combine else out
 
 
-def moe_experts(h: torch.Tensor, routing: MoeRouting, w_gate: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
-                activation: str = "silu") -> torch.Tensor:
-    """The weighted sum of the chosen experts' gated units, float32 ``[tokens, width]``.  ``w_gate`` and
-    ``w_up`` are ``[experts, ff, width]``, ``w_down`` ``[experts, width, ff]``, all in the type of ``h``."""
+def moe_experts(h: torch.Tensor, routing: MoeRouting, w_gate: torch.Tensor | None, w_up: torch.Tensor, w_down: torch.Tensor,
+                activation: str = "silu", combine: bool = True):
+    """The weighted sum of the chosen experts' units, float32 ``[tokens, width]`` (``combine=False``: the
+    :class:`WeightedRows` in front of the sum).  ``w_gate`` (``None``: ungated units) and ``w_up`` are ``[experts, ff,
+    width]``, ``w_down`` ``[experts, width, ff]``, all in the type of ``h``."""
     n, width = h.shape
-    experts, ff, _ = w_gate.shape
+    experts, ff, _ = w_up.shape
     top = routing.chosen.shape[1]
+    gated = w_gate is not None
     for name, t, shape in (("w_gate", w_gate, (experts, ff, width)), ("w_up", w_up, (experts, ff, width)),
                            ("w_down", w_down, (experts, width, ff))):
+        if t is None:
+            continue
         _want(t, h.dtype, name)
         if t.shape != shape:
             raise KernelError(f"{name} must be {shape}")
+    act_code = _moe_activation(activation, gated)
     pairs = n * top
     act = torch.empty((pairs, ff), dtype=h.dtype, device=h.device)
     y = torch.empty((pairs, width), dtype=torch.float32, device=h.device)
-    out = torch.empty((n, width), dtype=torch.float32, device=h.device)
     lib, r = _lib(), routing
-    _check(lib.tk_moe_ffn(h.data_ptr(), h.stride(0), top, w_gate.data_ptr(), w_up.data_ptr(), act.data_ptr(),
+    first, second = (w_gate, w_up) if gated else (w_up, None)
+    _check(lib.tk_moe_ffn(h.data_ptr(), h.stride(0), top, first.data_ptr(), _ptr(second), act.data_ptr(),
                           r.order.data_ptr(), r.tiles.data_ptr(), r.n_tiles.data_ptr(), r.max_tiles, ff, width,
-                          GLU_ACTIVATIONS[activation], dtype_code(h.dtype), _stream()), "moe_ffn (gate, up)")
+                          act_code, MOE_GATED if gated else MOE_UNARY, dtype_code(h.dtype), _stream()),
+           "moe_ffn (first product)")
     _check(lib.tk_moe_ffn(act.data_ptr(), ff, 1, w_down.data_ptr(), None, y.data_ptr(), r.order.data_ptr(),
-                          r.tiles.data_ptr(), r.n_tiles.data_ptr(), r.max_tiles, width, ff, 0, dtype_code(h.dtype),
-                          _stream()), "moe_ffn (down)")
-    _check(lib.tk_moe_combine(y.data_ptr(), r.weights.data_ptr(), out.data_ptr(), n, width, top, _stream()),
-           "moe_combine")
-    return out
+                          r.tiles.data_ptr(), r.n_tiles.data_ptr(), r.max_tiles, width, ff, 0, MOE_SUMS,
+                          dtype_code(h.dtype), _stream()), "moe_ffn (down)")
+    out = WeightedRows(y, r.weights, None)
+    return out.combine() if combine else out
 
 
 def decode_splits(n_items: int, n_kv_heads: int, max_kv_len: int) -> int:
@@ -1551,14 +1671,14 @@ def latent_prepare(proj: torch.Tensor, cache: torch.Tensor, positions: torch.Ten
                    req_slot: torch.Tensor, block_table: torch.Tensor, err: torch.Tensor, *, kv_off: int, rank: int,
                    rot: int, kv_norm_w: torch.Tensor, eps: float, table: torch.Tensor | None = None,
                    q_abs: torch.Tensor | None = None, q_off: int = 0, q_head_cols: int = 0, q_rot_off: int = 0,
-                   cq_off: int = 0, cq_norm_w: torch.Tensor | None = None,
+                   cq_off: int = 0, cq_norm_w: torch.Tensor | None = None, halves: bool = False,
                    req_q_len: torch.Tensor | None = None, req_kv_len: torch.Tensor | None = None):
     """A latent cache's rows for the step's tokens, and what the queries need, from the columns of the
     stacked projection ``proj`` (the cache's type, or float32 partial sums).
 
     Columns ``kv_off .. + rank`` are RMS-normed with ``kv_norm_w`` (the latent), the ``rot`` columns
     behind them are the shared key part, whose first ``2 * table.shape[1]`` elements turn as
-    neighbouring pairs by the (cos, sin) of ``table``; both go to the token's row of ``cache``
+    neighbouring pairs (``halves``: as pairs half of them apart) by the (cos, sin) of ``table``; both go to the token's row of ``cache``
     ``[pages, 1, page, rank + rot]``.  With ``q_abs`` (float32 ``[heads, tokens, rank]``) the query rows
     ``[tokens, heads, rank + rot]`` are returned in float32: ``q_abs`` and the turned columns
     ``q_off + h * q_head_cols + q_rot_off .. + rot``.  With ``cq_norm_w`` the columns ``cq_off .. +
@@ -1595,9 +1715,9 @@ def latent_prepare(proj: torch.Tensor, cache: torch.Tensor, positions: torch.Ten
                                        cq_rank, kv_norm_w.data_ptr(), _ptr(cq_norm_w), _ptr(cq), _ptr(q_abs), _ptr(q_lat),
                                        cache.data_ptr(), _ptr(table), positions.data_ptr(), tok_req.data_ptr(),
                                        req_slot.data_ptr(), block_table.data_ptr(), _ptr(req_q_len), _ptr(req_kv_len),
-                                       err.data_ptr(), n, req_slot.numel(), heads, rank, rot, pairs, page_size,
-                                       block_table.shape[1], num_pages, float(eps), dtype_code(cache.dtype), _stream()),
-           "latent_prepare")
+                                       err.data_ptr(), n, req_slot.numel(), heads, rank, rot, pairs, int(bool(halves)),
+                                       page_size, block_table.shape[1], num_pages, float(eps), dtype_code(cache.dtype),
+                                       _stream()), "latent_prepare")
     return q_lat, cq
 
 

@@ -23,6 +23,16 @@ __device__ __forceinline__ float stacked_ld(const StackedInput& in, size_t off) 
   return acc;
 }
 
+// Four neighbouring elements as float32 (the address is a multiple of four elements).
+template <typename T> __device__ __forceinline__ float4 ld4(const T* src);
+template <> __device__ __forceinline__ float4 ld4<float>(const float* src) { return *reinterpret_cast<const float4*>(src); }
+template <> __device__ __forceinline__ float4 ld4<__nv_bfloat16>(const __nv_bfloat16* src) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(src);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 // Four neighbouring values (the offset is a multiple of four elements), and the store of four.
 template <typename T> __device__ __forceinline__ float4 stacked_ld4(const StackedInput& in, size_t off);
 template <> __device__ __forceinline__ float4 stacked_ld4<float>(const StackedInput& in, size_t off) {

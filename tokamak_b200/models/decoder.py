@@ -7,8 +7,22 @@ from dataclasses import dataclass
 import torch
 
 from ..parts import embedding as _builtin_embedding   # registers the built-in embedding and head
-from ..parts.base import (BLOCKS, EMBEDDINGS, HEADS, NORMS, POSITIONS, OwedNorm, Runtime, TensorReq, graph_safe,
-                          weight_bytes)
+from ..parts.base import (BLOCKS, EMBEDDINGS, HEADS, NORMS, POSITIONS, OwedNorm, Runtime, SumBranch, TensorReq,
+                          graph_safe, weight_bytes)
+
+
+EMBEDDING_CACHE = "embedding"       # the cache key of an embedding that keeps something between steps
+
+
+@dataclass(frozen=True)
+class StreamInput:
+    """What joins the residual stream right before a call of the schedule, beside what the block before it left:
+    the embedded rows once more (``embedding``, as they were before the first block) and row ``row`` of the float32
+    vectors ``[rows, width]`` named ``table`` (one of the model's ``stream_tables``), the same for every token."""
+
+    embedding: bool = False
+    table: str | None = None
+    row: int = 0
 
 
 @dataclass(frozen=True)
@@ -18,11 +32,12 @@ class LayerCall:
     Naming a block twice runs its weights twice; two calls that name the same
     ``cache`` share keys and values (the later one must be built without key and
     value projections of its own).  ``cache`` is ``None`` for a block that keeps
-    nothing between steps.
+    nothing between steps.  ``joins`` says what else joins the stream before the block reads it.
     """
 
     block: str
     cache: str | None
+    joins: StreamInput | None = None
 
 
 @dataclass(frozen=True)
@@ -32,7 +47,8 @@ class ModelSpec:
     encoding that is added to the embedded rows (``None``: the mixers carry the positions).
     ``streams > 1``: the residual stream is kept in that many float32 copies ``[streams, tokens, width]``, all
     equal to the embedded rows at the start; the blocks and the last norm must know such a stream (the
-    ``hyper`` block, the ``layernorm`` norm, which reads the sum of the copies at the end)."""
+    ``hyper`` block, the ``layernorm`` norm, which reads the sum of the copies at the end).  ``stream_tables``:
+    ``(tensor name, rows)`` of the vectors that calls of the schedule add to the stream (``StreamInput``)."""
 
     embedding: object                  # an embedding spec (vocab_size, hidden_size, kind, ...)
     blocks: tuple                      # block specs, each with a unique ``name``
@@ -42,6 +58,7 @@ class ModelSpec:
     head: object                       # a head spec (vocab_size, kind, ...)
     embedding_position: object = None
     streams: int = 1
+    stream_tables: tuple = ()
 
     def __post_init__(self) -> None:
         names = [b.name for b in self.blocks]
@@ -50,6 +67,14 @@ class ModelSpec:
         for call in self.schedule:
             if call.block not in names:
                 raise ValueError(f"the schedule names an unknown block {call.block!r}")
+            if call.cache == EMBEDDING_CACHE:
+                raise ValueError(f"the cache key {EMBEDDING_CACHE!r} is the embedding's")
+            if call.joins is not None:
+                if self.streams > 1:
+                    raise ValueError("nothing else joins a stream that is kept in several copies")
+                rows = dict(self.stream_tables).get(call.joins.table, 0)
+                if call.joins.table is not None and not 0 <= call.joins.row < rows:
+                    raise ValueError(f"the model's stream tables have no row {call.joins.row} of {call.joins.table!r}")
 
 
 def flat_needs(key, need) -> list[tuple]:
@@ -88,6 +113,9 @@ class DecoderModel:
                                                           tensors, rt)
         self.head = HEADS.get(spec.head.kind)(spec.head, self.embedding, tensors, rt)
         self._needs = {name: block.cache_need() for name, block in self.blocks.items()}
+        self._embedding_need = self.embedding.cache_need() if hasattr(self.embedding, "cache_need") else None
+        self.stream_tables = {name: tensors[name].float().contiguous() for name, _ in spec.stream_tables}
+        self._keeps_embedding = any(call.joins is not None and call.joins.embedding for call in spec.schedule)
 
     @staticmethod
     def expected_tensors(spec: ModelSpec) -> dict[str, TensorReq]:
@@ -100,6 +128,8 @@ class DecoderModel:
             out.update(BLOCKS.get(b.kind).expected_tensors(b))
         out.update(NORMS.get(spec.final_norm.kind).expected_tensors(spec.final_norm,
                                                                     spec.final_norm_name))
+        for name, rows in spec.stream_tables:
+            out[name] = TensorReq((rows, spec.embedding.hidden_size), role="bias")
         out.update(HEADS.get(spec.head.kind).expected_tensors(spec.head))
         return out
 
@@ -121,7 +151,7 @@ class DecoderModel:
 
     def cache_needs(self) -> dict[str, object]:
         """Cache key -> need, checked for agreement between calls that share a key."""
-        needs: dict[str, object] = {}
+        needs: dict[str, object] = dict(flat_needs(EMBEDDING_CACHE, self._embedding_need))
         for call in self.spec.schedule:
             need = self.blocks[call.block].cache_need()
             if need is None:
@@ -136,11 +166,40 @@ class DecoderModel:
                 needs.setdefault(key, sub)
         return needs
 
-    def forward(self, step) -> torch.Tensor:
-        """Float32 logits ``[len(step.logits_rows), vocab]`` for the rows asked for."""
-        resid = self.embedding.forward(step)
+    def _embed(self, step) -> tuple[torch.Tensor, torch.Tensor | None]:
+        """The embedded rows and, where a call of the schedule adds them once more, a copy of them."""
+        kw, keep = {}, None
+        if self._embedding_need is not None:
+            kw["cache_view"] = views_of(step.cache, EMBEDDING_CACHE, self._embedding_need)
+        if self._keeps_embedding and self.embedding_position is None and getattr(self.embedding, "TAKES_KEEP", False):
+            keep = kw["keep"] = torch.empty((step.n_tokens, self.spec.embedding.hidden_size), dtype=torch.float32,
+                                            device=self.rt.device)
+        resid = self.embedding.forward(step, **kw)
         if self.embedding_position is not None:
             self.embedding_position.add_to_embedding(resid, step)
+        if self._keeps_embedding and keep is None:
+            keep = resid.clone()
+        return resid, keep
+
+    def _join(self, resid, pending, joins: StreamInput | None, embedded, norm):
+        """What ``norm`` finds pending: the branch that is waiting together with what ``joins`` names.  A norm that
+        adds it all in its own kernel gets a :class:`SumBranch`; in front of any other the rest is added here."""
+        if joins is not None:
+            extra = embedded if joins.embedding else None
+            vector = self.stream_tables[joins.table][joins.row] if joins.table is not None else None
+            if pending is None or isinstance(pending, (torch.Tensor, SumBranch)):
+                terms = pending.terms if isinstance(pending, SumBranch) else (() if pending is None else (pending,))
+                pending = SumBranch(terms, extra, vector)
+            else:
+                SumBranch((), extra, vector).settle(resid)      # the branch joins later; the sum is the same
+        if isinstance(pending, SumBranch) and not getattr(norm, "TAKES_SUM", False):
+            pending.settle(resid)
+            pending = None
+        return pending
+
+    def forward(self, step) -> torch.Tensor:
+        """Float32 logits ``[len(step.logits_rows), vocab]`` for the rows asked for."""
+        resid, embedded = self._embed(step)
         if self.spec.streams > 1:
             resid = resid.unsqueeze(0).repeat(self.spec.streams, 1, 1)
         pending = None
@@ -148,15 +207,20 @@ class DecoderModel:
         for i, call in enumerate(schedule):
             view = views_of(step.cache, call.cache, self._needs[call.block]) if call.cache is not None else None
             block = self.blocks[call.block]
+            pending = self._join(resid, pending, call.joins, embedded, getattr(block, "entry_norm", None))
             if getattr(block, "TAKES_NEXT_NORM", False):
-                # the norm that will consume what the block leaves pending: the next block's, or the last
+                # the norm that will consume what the block leaves pending: the next block's, or the last; none
+                # where more joins the stream before it
                 after = self.blocks[schedule[i + 1].block] if i + 1 < len(schedule) else None
                 next_norm = getattr(after, "entry_norm", None) if after is not None else self.final_norm
+                if after is not None and schedule[i + 1].joins is not None:
+                    next_norm = None
                 resid, pending = block.forward(resid, pending, step, view, next_norm=next_norm)
             else:
                 resid, pending = block.forward(resid, pending, step, view)
         if step.n_want == 0:
             return torch.empty((0, self.spec.head.vocab_size), dtype=torch.float32, device=resid.device)
+        pending = self._join(resid, pending, None, None, self.final_norm)
         # every request brings one token and wants it: the wanted rows are all rows, in order
         all_rows = step.n_want == step.n_tokens and step.max_q_len == 1
         h = self.final_norm.add_norm(resid, pending, rows=None if all_rows and isinstance(pending, OwedNorm) else step.logits_rows)

@@ -25,7 +25,8 @@ feed_forward   ``expected_tensors(spec, prefix)``, ``__init__(spec, prefix, tens
 block          ``expected_tensors(spec)``, ``__init__(spec, tensors, rt)``,
                ``cache_need()``, ``forward(resid, pending, step, cache_view) -> (resid, pending)``
 embedding      ``expected_tensors(spec)``, ``__init__(spec, tensors, rt)``,
-               ``forward(step) -> float32 residual rows [N, hidden]``, attribute ``weight``
+               ``forward(step) -> float32 residual rows [N, hidden]``, attribute ``weight``; one that keeps
+               something between steps has ``cache_need()`` and takes ``forward(step, cache_view=)``
 head           ``expected_tensors(spec)``, ``__init__(spec, embedding part, tensors, rt)``,
                ``forward(h, step) -> float32 logits [rows, vocab]``
 =============  ==========================================================
@@ -78,6 +79,14 @@ norm a float32 tensor ``[streams, N, hidden]`` instead of ``[N, hidden]``.  A bl
 :class:`HyperBranch` pending (the sublayer's output with the weights of its write to every copy); a norm that
 knows it (``layernorm``) takes ``add_norm(resid, pending, rows, read=)`` and does the write, the weighted read and
 the norm in one kernel.
+
+**Several branches at once.**  A block whose sublayers read the same input side by side, and a schedule in which
+something else joins the stream between two blocks (:class:`~tokamak_b200.models.decoder.StreamInput`), leave a
+:class:`SumBranch` pending.  A norm with ``TAKES_SUM = True`` adds all of it to the stream and normalises in one
+kernel; in front of any other norm the model adds it first (:meth:`SumBranch.settle`).  A feed-forward with
+``LEAVES_WEIGHTED_ROWS = True`` takes ``combine=False`` and may return
+:class:`~tokamak_b200.csrc.ops.WeightedRows` (a mixture's rows before their weighted sum), which can be a term of a
+``SumBranch``.  An embedding with ``TAKES_KEEP = True`` takes ``keep=``, a float32 tensor for a second copy of its rows.
 
 ``TAKES_PROJ = True`` (a mixer that can be half of a ``parallel`` mixer): its stacked input projection is ``w_in``
 and its ``branch`` takes ``proj=, proj_off=``, a product of the shared input that holds its columns from
@@ -221,6 +230,26 @@ class HyperBranch:
     mix: torch.Tensor | None = None
     write: torch.Tensor | None = None
     mult: float = 1.0
+
+
+@dataclass
+class SumBranch:
+    """Everything that waits to join the residual stream at one place: the outputs of sublayers that ran side by
+    side (``terms``: what :func:`linear` returned, or ``WeightedRows``), float32 rows like the stream's (``extra``)
+    and one float32 vector for every token (``vector``), all added in 32-bit."""
+
+    terms: tuple = ()
+    extra: torch.Tensor | None = None
+    vector: torch.Tensor | None = None
+
+    def settle(self, resid: torch.Tensor) -> None:
+        """Add everything to the stream (for a norm that does not do so itself)."""
+        from ..csrc import ops
+        for term in self.terms:
+            resid.add_(term.combine() if isinstance(term, ops.WeightedRows) else sum_parts(term, torch.float32))
+        for term in (self.extra, self.vector):
+            if term is not None:
+                resid.add_(term)
 
 
 @dataclass

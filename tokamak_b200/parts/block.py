@@ -6,8 +6,8 @@ from dataclasses import dataclass
 
 import torch
 
-from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, HyperBranch, NormedBranch, OwedNorm, Runtime, TensorReq,
-                   graph_safe, weight_bytes)
+from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, HyperBranch, NormedBranch, OwedNorm, Runtime, SumBranch,
+                   TensorReq, graph_safe, weight_bytes)
 
 
 @dataclass(frozen=True)
@@ -368,3 +368,74 @@ class HyperBlock:
             h = self.norm2.add_norm(resid, pending, read=read)
             pending = HyperBranch(self.feed_forward.forward(h, step), mix, write, self.spec.mult)
         return resid, pending
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """A block whose mixer and feed-forward (which may be absent) read the output of one norm side by side.
+    ``norm1_name`` is a full tensor name; the prefixes end with a dot."""
+
+    name: str
+    norm1: object
+    mixer: object
+    norm1_name: str
+    mixer_prefix: str
+    feed_forward: object = None
+    ffn_prefix: str | None = None
+    kind: str = "parallel"
+
+
+@BLOCKS.register("parallel")
+class ParallelBlock:
+    """``h = norm1(x)``, ``x <- x + (mixer(h) + ff(h))``.
+
+    Both outputs are left pending as one :class:`~tokamak_b200.parts.base.SumBranch`; the norm of the next block (or
+    the model's last) adds them to the float32 stream and normalises the sum in one kernel.  A mixture of
+    experts leaves its rows in front of their weighted sum, which that kernel forms too."""
+
+    def __init__(self, spec: ParallelBlockSpec, tensors: dict[str, torch.Tensor], rt: Runtime):
+        self.spec = spec
+        self.norm1 = NORMS.get(spec.norm1.kind)(spec.norm1, spec.norm1_name, tensors, rt)
+        self.mixer = MIXERS.get(spec.mixer.kind)(spec.mixer, spec.mixer_prefix, tensors, rt)
+        self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward = FEED_FORWARDS.get(spec.feed_forward.kind)(spec.feed_forward, spec.ffn_prefix, tensors, rt)
+
+    @staticmethod
+    def expected_tensors(spec: ParallelBlockSpec) -> dict[str, TensorReq]:
+        out: dict[str, TensorReq] = {}
+        out.update(NORMS.get(spec.norm1.kind).expected_tensors(spec.norm1, spec.norm1_name))
+        out.update(MIXERS.get(spec.mixer.kind).expected_tensors(spec.mixer, spec.mixer_prefix))
+        if spec.feed_forward is not None:
+            out.update(FEED_FORWARDS.get(spec.feed_forward.kind).expected_tensors(spec.feed_forward, spec.ffn_prefix))
+        return out
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def _parts(self) -> list:
+        return [p for p in (self.norm1, self.mixer, self.feed_forward) if p is not None]
+
+    def GRAPH_SAFE(self) -> bool:
+        return graph_safe(*self._parts())
+
+    @property
+    def prefill_heads(self) -> int | None:
+        return getattr(self.mixer, "prefill_heads", None)
+
+    def weight_bytes(self) -> int:
+        return weight_bytes(*self._parts())
+
+    @property
+    def entry_norm(self):
+        return self.norm1
+
+    def forward(self, resid: torch.Tensor, pending, step, cache_view):
+        h = self.norm1.add_norm(resid, pending)
+        if isinstance(h, OwedNorm):
+            h = h.materialize()
+        terms = [self.mixer.forward(h, step, cache_view)]
+        if self.feed_forward is not None:
+            kw = {"combine": False} if getattr(self.feed_forward, "LEAVES_WEIGHTED_ROWS", False) else {}
+            terms.append(self.feed_forward.forward(h, step, **kw))
+        return resid, SumBranch(tuple(terms))

@@ -6,6 +6,7 @@ from dataclasses import dataclass
 
 import torch
 
+from ..cache.manager import StateNeed
 from ..csrc import ops
 from .base import EMBEDDINGS, HEADS, Runtime, TensorReq, chain_of, linear, sum_parts, tensor_bytes
 
@@ -33,6 +34,23 @@ class HeadSpec:
     softcap: float | None = None    # and then bounded: cap * tanh(logits / cap)
 
 
+@dataclass(frozen=True)
+class BigramEmbeddingSpec:
+    """A token table and a table of ``buckets + 1`` rows by hashed pairs: a token's row is ``scale * table[id]`` plus
+    the pair row ``(previous id * mul_prev + id * mul_cur) mod buckets``, or the last pair row for a request's first
+    token."""
+
+    vocab_size: int
+    hidden_size: int
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+    name: str = "embed"
+    pair_name: str = "bigram"
+    scale: float = 1.0
+    kind: str = "embedding_bigram"
+
+
 @EMBEDDINGS.register("embedding")
 class Embedding:
     """Row lookup (src/tokamak/model/transformer.py:140), times the spec's ``scale`` where a
@@ -55,6 +73,38 @@ class Embedding:
         resid = torch.empty((step.n_tokens, self.spec.hidden_size), dtype=torch.float32,
                             device=self.weight.device)
         ops.embed_gather(self.weight, step.token_ids, resid, step.err, scale=self.spec.scale)
+        return resid
+
+
+@EMBEDDINGS.register("embedding_bigram")
+class BigramEmbedding:
+    """Two row lookups added in float32.  A request's last token is part of its state (one int32 record a slot):
+    the next step's first token of the request forms its pair with it."""
+
+    GRAPH_SAFE = True
+    TAKES_KEEP = True
+
+    def weight_bytes(self) -> int:
+        return 0          # read by row
+
+    def __init__(self, spec: BigramEmbeddingSpec, tensors: dict[str, torch.Tensor], rt: Runtime):
+        self.spec = spec
+        self.weight = tensors[spec.name]
+        self.pairs = tensors[spec.pair_name]
+
+    @staticmethod
+    def expected_tensors(spec: BigramEmbeddingSpec) -> dict[str, TensorReq]:
+        return {spec.name: TensorReq((spec.vocab_size, spec.hidden_size)),
+                spec.pair_name: TensorReq((spec.buckets + 1, spec.hidden_size))}
+
+    def cache_need(self) -> StateNeed:
+        return StateNeed((1,), "int32")
+
+    def forward(self, step, cache_view, keep: torch.Tensor | None = None) -> torch.Tensor:
+        s = self.spec
+        resid = torch.empty((step.n_tokens, s.hidden_size), dtype=torch.float32, device=self.weight.device)
+        ops.embed_bigram(self.weight, self.pairs, cache_view.records, step, resid, mul_prev=s.mul_prev, mul_cur=s.mul_cur,
+                         scale=s.scale, keep=keep)
         return resid
 
 

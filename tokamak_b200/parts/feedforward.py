@@ -158,8 +158,10 @@ class Mlp:
 
 @dataclass(frozen=True)
 class MoESpec:
-    """A mixture of ``num_experts`` gated units of inner size ``intermediate_size`` of which every token uses
-    ``top``.  The experts form ``num_groups`` equal groups of neighbours and only experts of the ``keep_groups``
+    """A mixture of ``num_experts`` units of inner size ``intermediate_size`` of which every token uses ``top``.
+    ``gated``: a unit is ``down(act(gate(x)) * up(x))`` with ``activation`` ``silu`` or ``gelu_tanh``; otherwise
+    ``down(act(up(x)))`` with ``relu2``, ``silu`` or ``gelu_tanh``.  ``router``: ``sigmoid`` (the weights are the chosen
+    experts' plain scores) or ``softmax`` (the softmax over the chosen experts' logits only).  The experts form ``num_groups`` equal groups of neighbours and only experts of the ``keep_groups``
     best groups can be chosen (``num_groups = keep_groups = 1``: no restriction).  ``correction``: a learned
     number per expert that is added to the scores for the choice only.  The ``*_name`` fields are the
     tensors' names after the part's prefix; expert ``e``'s matrices lie under ``expert_prefix.format(e)``."""
@@ -171,6 +173,8 @@ class MoESpec:
     num_groups: int = 1
     keep_groups: int = 1
     correction: bool = True
+    gated: bool = True
+    router: str = "sigmoid"
     activation: str = "silu"
     router_name: str = "router"
     correction_name: str = "correction"
@@ -186,8 +190,10 @@ class MixtureOfExperts:
     """Router scores are sigmoids of 32-bit logits, ``s = sigmoid(W_r h)``; the choice is made on
     ``s + correction``: a group's score is the sum of its two largest choice scores, experts outside the best
     groups cannot be chosen, and the ``top`` largest of the rest are; the weights are the chosen experts'
-    plain scores, not renormalised; the output is the weighted sum of the chosen experts'
-    ``W_down (act(W_gate h) * (W_up h))``.  Experts have no biases.
+    plain scores, not renormalised.  A softmax router chooses on the 32-bit logits (plus ``correction``) in the
+    same way, and its weights are the softmax over the chosen experts' logits only.  The output is the weighted sum
+    of the chosen experts' ``W_down (act(W_gate h) * (W_up h))``, or ``W_down act(W_up h)`` for ungated ones.
+    Experts have no biases.
 
     The experts' matrices are stacked ``[experts, ...]`` at load.  A step's (token, choice) pairs are laid
     out expert by expert on the device, so nothing is read back and a step of single tokens can be
@@ -196,10 +202,14 @@ class MixtureOfExperts:
     """
 
     GRAPH_SAFE = True
+    LEAVES_WEIGHTED_ROWS = True
 
     def __init__(self, spec: MoESpec, prefix: str, tensors: dict[str, torch.Tensor], rt: Runtime):
-        if spec.activation not in ops.GLU_ACTIVATIONS:
-            raise ValueError(f"unknown activation {spec.activation!r}; known: {', '.join(ops.GLU_ACTIVATIONS)}")
+        known = ops.GLU_ACTIVATIONS if spec.gated else ops.UNARY_ACTIVATIONS
+        if spec.activation not in known:
+            raise ValueError(f"unknown activation {spec.activation!r}; known: {', '.join(known)}")
+        if spec.router not in ops.ROUTER_KINDS:
+            raise ValueError(f"unknown router {spec.router!r}; known: {', '.join(ops.ROUTER_KINDS)}")
         if spec.num_experts % spec.num_groups or not 1 <= spec.keep_groups <= spec.num_groups:
             raise ValueError(f"{spec.num_experts} experts do not form {spec.num_groups} equal groups of which "
                              f"{spec.keep_groups} are kept")
@@ -212,12 +222,14 @@ class MixtureOfExperts:
         self.correction = tensors[prefix + spec.correction_name].contiguous() if spec.correction else None
         stack = lambda name: torch.stack([tensors[prefix + spec.expert_prefix.format(e) + name]
                                           for e in range(spec.num_experts)]).contiguous()
-        self.w_gate, self.w_up, self.w_down = stack(spec.gate_name), stack(spec.up_name), stack(spec.down_name)
+        self.w_gate = stack(spec.gate_name) if spec.gated else None
+        self.w_up, self.w_down = stack(spec.up_name), stack(spec.down_name)
         # bfloat16 at sizes the product on pairs of SMs takes: gate and up rows alternate in blocks, so that
-        # the activation is the product's epilogue; the two matrices are then kept only in that form
-        self.w_gate_up = None
-        if ops.moe_tc_takes(self.w_gate.dtype, spec.hidden_size, spec.intermediate_size):
-            self.w_gate_up = ops.moe_stack_gate_up(self.w_gate, self.w_up)
+        # the activation is the product's epilogue (an ungated unit's first matrix is taken as it is); the
+        # matrices are then kept only in that form
+        self.w_first = None
+        if ops.moe_tc_takes(self.w_up.dtype, spec.hidden_size, spec.intermediate_size, spec.gated):
+            self.w_first = ops.moe_stack_gate_up(self.w_gate, self.w_up) if spec.gated else self.w_up
             self.w_gate = self.w_up = None
 
     @staticmethod
@@ -226,7 +238,8 @@ class MixtureOfExperts:
         out = {}
         for e in range(spec.num_experts):
             p = prefix + spec.expert_prefix.format(e)
-            out[p + spec.gate_name] = TensorReq((i, h))
+            if spec.gated:
+                out[p + spec.gate_name] = TensorReq((i, h))
             out[p + spec.up_name] = TensorReq((i, h))
             out[p + spec.down_name] = TensorReq((h, i))
         out[prefix + spec.router_name] = TensorReq((spec.num_experts, h), role="matrix_f32")
@@ -236,20 +249,22 @@ class MixtureOfExperts:
 
     def weight_bytes(self) -> int:
         """What a step of one token reads: the router and ``top`` experts (a large step reads all)."""
-        per_expert = tensor_bytes(self.w_gate, self.w_up, self.w_gate_up, self.w_down) // self.spec.num_experts
+        per_expert = tensor_bytes(self.w_gate, self.w_up, self.w_first, self.w_down) // self.spec.num_experts
         return tensor_bytes(self.router, self.correction) + self.spec.top * per_expert
 
-    def forward(self, h, step):
+    def forward(self, h, step, combine: bool = True):
         spec = self.spec
         if isinstance(h, OwedNorm):
             h = h.materialize()
-        tc = self.w_gate_up is not None
+        tc = self.w_first is not None
         routing = ops.moe_route(h, self.router, self.correction, top=spec.top, n_groups=spec.num_groups,
-                                keep=spec.keep_groups, padded=tc)
-        if tc and ops.moe_small_takes(h.shape[0], spec.top, spec.hidden_size, spec.intermediate_size):
-            out = ops.moe_experts_small(h, routing, self.w_gate_up, self.w_down, activation=spec.activation)
+                                keep=spec.keep_groups, padded=tc, kind=spec.router)
+        kw = dict(activation=spec.activation, combine=combine)
+        if tc and ops.moe_small_takes(h.shape[0], spec.top, spec.hidden_size, spec.intermediate_size, spec.gated):
+            out = ops.moe_experts_small(h, routing, self.w_first, self.w_down, gated=spec.gated, **kw)
         elif tc:
-            out = ops.moe_experts_tc(h, routing, self.w_gate_up, self.w_down, step.err, activation=spec.activation)
+            out = ops.moe_experts_tc(h, routing, self.w_first, self.w_down, step.err, gated=spec.gated, **kw)
         else:
-            out = ops.moe_experts(h, routing, self.w_gate, self.w_up, self.w_down, activation=spec.activation)
-        return out.unsqueeze(0)         # float32 sums, one part: the consuming norm reads them as they are
+            out = ops.moe_experts(h, routing, self.w_gate, self.w_up, self.w_down, **kw)
+        # float32 sums, one part: the consuming norm reads them as they are
+        return out.unsqueeze(0) if combine else out

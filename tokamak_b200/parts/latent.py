@@ -21,8 +21,8 @@ class LatentAttentionSpec:
     A head has ``head_dim`` unrotated and ``rot_dim`` rotated query/key elements and ``v_head_dim``
     value elements; ``kv_rank`` is the size of the cached latent.  ``q_rank`` (``None``: the queries
     are a direct projection) is the size of a latent that the queries pass through, with a norm of
-    its own.  ``position`` rotates the ``rot_dim`` part (a spec whose part rotates neighbouring pairs,
-    or none).  ``window``: positions a query sees, itself included (``None``: all).  ``sinks``: a learned
+    its own.  ``position`` rotates the ``rot_dim`` part (a spec whose part rotates neighbouring pairs
+    or halves, or none).  ``window``: positions a query sees, itself included (``None``: all).  ``sinks``: a learned
     number per head joins the softmax denominator.  ``gate``: the concatenated heads are multiplied by
     the sigmoid of a projection of the mixer's input.  ``norm_eps`` is the eps of the latents' norms.
     """
@@ -93,8 +93,10 @@ class LatentAttention:
         self.sinks = t(spec.sink_name).contiguous() if spec.sinks else None
         self.w_o = t(spec.o_name)
         self.position = POSITIONS.get(spec.position.kind)(spec.position, tensors, rt)
-        if dr and spec.position.kind != "none" and getattr(self.position, "PAIRING", None) != "neighbours":
-            raise ValueError(f"position encoding {spec.position.kind!r} does not rotate neighbouring pairs")
+        pairing = getattr(self.position, "PAIRING", None)
+        if dr and spec.position.kind != "none" and pairing not in ("neighbours", "halves"):
+            raise ValueError(f"position encoding {spec.position.kind!r} rotates neither neighbouring pairs nor halves")
+        self.halves = pairing == "halves"
 
     @staticmethod
     def expected_tensors(spec: LatentAttentionSpec, prefix: str) -> dict[str, TensorReq]:
@@ -145,7 +147,7 @@ class LatentAttention:
         proj = linear(h, self.w_in, err=step.err)
         table, _ = self.position.rotary_table(step)
         prepare = dict(kv_off=self.kv_off, rank=r, rot=dr, kv_norm_w=self.kv_norm_w, eps=spec.norm_eps, table=table,
-                       req_q_len=step.req_q_len, req_kv_len=step.req_kv_len)
+                       halves=self.halves, req_q_len=step.req_q_len, req_kv_len=step.req_kv_len)
         where = (cache_view.k, step.positions, step.tok_req, step.req_slot, cache_view.table, step.err)
         if spec.q_rank:
             # the kernel that writes the cache rows also norms the query latent; its up-projection follows

@@ -7,7 +7,7 @@ from dataclasses import dataclass
 import torch
 
 from ..csrc import ops
-from .base import NORMS, HyperBranch, NormedBranch, OwedNorm, Runtime, TensorReq
+from .base import NORMS, HyperBranch, NormedBranch, OwedNorm, Runtime, SumBranch, TensorReq
 
 
 @dataclass(frozen=True)
@@ -27,6 +27,7 @@ class RMSNorm:
     """
 
     GRAPH_SAFE = True
+    TAKES_SUM = True           # a SumBranch joins in the same kernel
 
     def __init__(self, spec: RMSNormSpec, name: str, tensors: dict[str, torch.Tensor], rt: Runtime):
         self.spec = spec
@@ -52,13 +53,20 @@ class RMSNorm:
         normalised and ``resid`` is left as it is.  ``delta`` may be an
         :class:`OwedNorm`: the branch has been added to ``resid`` already; if it was
         prepared for this norm it is handed on as it is (its consumer pays the scale).
-        A :class:`NormedBranch` is normalised, scaled and added by the same kernel.
+        A :class:`NormedBranch` is normalised, scaled and added by the same kernel; all of a
+        :class:`SumBranch` joins in one.
         """
         if isinstance(delta, NormedBranch):
             n = rows.numel() if rows is not None else resid.shape[0]
             out = torch.empty((n, self.spec.dim), dtype=self.rt.dtype, device=resid.device)
             ops.branch_norm_add(resid, delta.x, delta.weight, delta.layer_scale, delta.eps, self.weight, out,
                                 self.spec.eps, rows, branch_groups=delta.groups)
+            return out
+        if isinstance(delta, SumBranch):
+            n = rows.numel() if rows is not None else resid.shape[0]
+            out = torch.empty((n, self.spec.dim), dtype=self.rt.dtype, device=resid.device)
+            ops.sum_rmsnorm(resid, delta.terms, out, self.weight, self.spec.eps, rows=rows, extra=delta.extra,
+                            vector=delta.vector)
             return out
         if isinstance(delta, OwedNorm):
             if delta.norm is self:
