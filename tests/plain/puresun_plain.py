@@ -93,9 +93,17 @@ def expert_ff(x, up, down, ROUND=no_round):
     return ROUND(ROUND(a * a) @ down.T)
 
 
-def mixture(h, w, mlp, ROUND=no_round):
-    T = h.shape[0]
+def choice_margin(h, router, top):
+    """[T] by how much the last chosen logit beats the first one that is not chosen."""
+    z = (h @ router.T).sort(-1, descending=True).values
+    return z[:, top - 1] - z[:, top] if top < z.shape[1] else torch.full((z.shape[0],), math.inf, dtype=z.dtype)
+
+
+def mixture(h, w, mlp, ROUND=no_round, margins_out=None):
+    """The weighted sum of the chosen experts' outputs."""
     idx, weight = route(h, w["router"], mlp["router"]["top"])
+    if margins_out is not None:
+        margins_out.append(choice_margin(h, w["router"], mlp["router"]["top"]))
     out = torch.zeros_like(h)
     for e in range(mlp["router"]["experts"]):
         t, k = torch.nonzero(idx == e, as_tuple=True)
@@ -121,19 +129,20 @@ def run_order(cfg):
     return order + [(i, None) for i in range(b, n)]
 
 
-def parallel_layer(x, cfg, lay, w, positions, ROUND=no_round):
+def parallel_layer(x, cfg, lay, w, positions, ROUND=no_round, margins_out=None):
     """x + (mixer(h) + ff(h)) with one norm in front of both."""
     eps = cfg["norm"]["eps"]
     h = ROUND(rms_norm(x, w["norm1"], eps))
     y = latent_attention(h, layer_weights(w, "mix."), lay["mixer"], eps, positions, ROUND)
     if lay.get("mlp") is not None:
-        y = y + mixture(h, layer_weights(w, "mlp."), lay["mlp"], ROUND)
+        y = y + mixture(h, layer_weights(w, "mlp."), lay["mlp"], ROUND, margins_out)
     return x + y
 
 
-def forward(cfg, weights, tokens, ROUND=no_round, layers_out=None):
+def forward(cfg, weights, tokens, ROUND=no_round, layers_out=None, margins_out=None):
     """Logits [T, vocab] of one sequence from position 0; ``weights`` maps names to float64 tensors.
-    ``layers_out``: a list that receives the residual stream after every layer run."""
+    ``layers_out``: a list that receives the residual stream after every layer run;
+    ``margins_out``: one that receives every router's margins."""
     positions = torch.arange(len(tokens))
     emb = embedding(weights, tokens, (cfg.get("embedding") or {}).get("bigram"))
     x = emb.clone()
@@ -142,7 +151,7 @@ def forward(cfg, weights, tokens, ROUND=no_round, layers_out=None):
             if p > 0:
                 x = x + emb
             x = x + weights["loop.step"][p]
-        x = parallel_layer(x, cfg, cfg["layers"][i], layer_weights(weights, f"l{i}."), positions, ROUND)
+        x = parallel_layer(x, cfg, cfg["layers"][i], layer_weights(weights, f"l{i}."), positions, ROUND, margins_out)
         if layers_out is not None:
             layers_out.append(x)
     logits = ROUND(rms_norm(x, weights["final.norm"], cfg["norm"]["eps"])) @ weights["head"].T
