@@ -1628,11 +1628,163 @@ def pukinex_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
     return rows
 
 
+# ------------------------------------------------------------------------------------------------
+# --design puresun: the Puresun design beside a Logivik model of latent attention layers of equal sizes (the
+# engine's other design with latent attention); its experts' kernels beside those of Tarivik's mixtures
+
+PURESUN_EXPERTS, PURESUN_TOP = 16, 2
+
+
+def puresun_config(s: dict) -> dict:
+    """Windowed latent attention (latents of 512, 64 rotated elements, heads of 128) beside a mixture of 16 ungated
+    experts of which 2 are used, together as wide as the twin's feed-forward, in every layer; two of the layers
+    run twice, so that there are as many layer runs as the twin has layers."""
+    d = s["dim"]
+    m = {"heads": s["heads"], "dim": d, "rot_dim": 64, "vdim": d, "kv_rank": 512, "scale": (d + 64) ** -0.5,
+         "mask": {"size": s["window"]}, "rot": {"base": 1e6, "dims": 64}}
+    mlp = {"kind": "moe", "expert": {"ff": s["ff"] // PURESUN_TOP}, "router": {"experts": PURESUN_EXPERTS, "top": PURESUN_TOP}}
+    layers = [{"type": "latent_attention", "mixer": m, "mlp": mlp} for _ in range(s["layers"] - 2)]
+    return {"architecture": "Puresun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}
+
+
+def logivik_latent_twin(s: dict) -> dict:
+    """A Logivik configuration whose layers are all windowed latent attention with a dense gated feed-forward."""
+    raw = logivik_config(s)
+    return dict(raw, layers=[raw["layers"][0]] * s["layers"])
+
+
+def puresun_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> list[dict]:
+    """Every kernel of the design alone, beside the like kernel of the Logivik or Tarivik path at the same shape:
+    time, achieved bytes or flops per second, and the fraction of the measured peak."""
+    import torch
+    from types import SimpleNamespace
+    from tokamak_b200.csrc import ops
+    dev = "cuda"
+    gen = torch.Generator(device=dev).manual_seed(0)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    err = torch.zeros(4, dtype=torch.int32, device=dev)
+    hq, d, page, win, width, vocab = s["heads"], s["dim"], 16, s["window"], s["width"], s["vocab"]
+    rank, rot, experts, top, ffe = 512, 64, PURESUN_EXPERTS, PURESUN_TOP, s["ff"] // PURESUN_TOP
+    bf = lambda *shape: torch.randn(shape, device=dev, generator=gen).bfloat16()
+    f32 = lambda *shape: torch.randn(shape, device=dev, generator=gen)
+    rows = []
+
+    def row(kernel, like, us, us_like, nbytes=0, flops=0.0, like_bytes=0, like_flops=0.0, note=""):
+        r = {"kernel": kernel, "like": like, "us": round(us, 1), "like_us": round(us_like, 1) if us_like else None}
+        for name, t, fl, nb in (("", us, flops, nbytes), ("like_", us_like, like_flops or flops, like_bytes or nbytes)):
+            if not t:
+                continue
+            if fl:
+                r[name + "bf16_frac"] = round(fl / (t * 1e-6) / 1e12 / peaks["bf16_tflops"], 4)
+            elif nb:
+                r[name + "hbm_frac"] = round(nb / (t * 1e-6) / 1e9 / peaks["hbm_gbs"], 4)
+        if note:
+            r["note"] = note
+        rows.append(r)
+
+    table_e, pairs = bf(vocab, width), bf(65522, width)
+    w_up, w_down = bf(experts, ffe, width) * width ** -0.5, bf(experts, width, ffe) * ffe ** -0.5
+    wgu = ops.moe_stack_gate_up(bf(experts, ffe, width) * width ** -0.5, w_up)
+    router, corr = f32(experts, width) * 0.05, f32(experts) * 0.05
+    w1 = torch.ones(width, device=dev)
+    freq = (1.0 / (1e6 ** (torch.arange(0, rot, 2, dtype=torch.float32) / rot))).to(dev)
+    for name, n, n_req, start in (("prompt", tokens, 1, 0), ("single tokens", batch, batch, ctx - 1)):
+        single = n_req > 1
+        t_us = lambda run, **kw: _time_us(run, graph=single, **kw)
+        per = n // n_req
+        step = SimpleNamespace(token_ids=torch.randint(0, vocab, (n,), device=dev, generator=gen, dtype=torch.int32),
+                               positions=i32([start + i for _ in range(n_req) for i in range(per)]),
+                               tok_req=i32([r for r in range(n_req) for _ in range(per)]),
+                               req_q_start=i32([r * per for r in range(n_req)]), req_q_len=i32([per] * n_req),
+                               req_kv_len=i32([start + per] * n_req), req_slot=i32(list(range(n_req))), err=err)
+        # ---- embedding
+        resid, keep, last = torch.empty(n, width, device=dev), torch.empty(n, width, device=dev), torch.zeros(n_req, 1, dtype=torch.int32, device=dev)
+        row(f"token rows + pair rows + the copy for the loop, {name}", f"token rows, {name}",
+            t_us(lambda: ops.embed_bigram(table_e, pairs, last, step, resid, mul_prev=31, mul_cur=17, keep=keep)),
+            t_us(lambda: ops.embed_gather(table_e, step.token_ids, resid, err)),
+            nbytes=n * width * (2 + 2 + 4 + 4), like_bytes=n * width * (2 + 4))
+        # ---- attention in the latent space
+        pages_req = -(-(start + per) // page)
+        table = torch.randperm(n_req * pages_req, device=dev, generator=gen).to(torch.int32).view(n_req, pages_req)
+        work = dict(items=i32(list(range(n)))) if single else dict(tiles=i32([x for t in reversed(range(-(-n // 64))) for x in (0, t)]))
+        if single:
+            work["n_splits"] = ops.latent_decode_splits(table.device, n, ctx, win)
+        keys = sum(min(start + i + 1, win) for _ in range(n_req) for i in range(per))
+
+        def attention(dr):
+            cache = bf(n_req * pages_req, 1, page, rank + dr) * 0.3
+            q = f32(n, hq, rank + dr) * 0.1
+            out = torch.empty(n, hq, rank, dtype=torch.bfloat16, device=dev)
+            return t_us(lambda: ops.attention_latent(q, out, cache, rank, step, table, scale=0.07, window=win, **work),
+                        iters=20 if single else 5)
+        kw = (dict(nbytes=keys * (rank + rot) * 2, like_bytes=keys * rank * 2) if single else
+              dict(flops=2.0 * keys * hq * (2 * rank + rot), like_flops=4.0 * keys * hq * rank))
+        row(f"latent attention (window, rotated part), {name}", f"latent attention (window), {name}", attention(rot), attention(0), **kw)
+        # ---- what stands around it
+        cols = hq * (d + rot) + rank + rot + hq * d
+        proj = bf(n, cols)
+        cache = torch.zeros(n_req * pages_req, 1, page, rank + rot, dtype=torch.bfloat16, device=dev)
+        rope, q_abs, ones_r = ops.rope_table(step.positions, freq), f32(hq, n, rank), torch.ones(rank, device=dev)
+        prep = lambda halves: ops.latent_prepare(proj, cache, step.positions, step.tok_req, step.req_slot, table, err,
+                                                 kv_off=hq * (d + rot), rank=rank, rot=rot, kv_norm_w=ones_r, eps=1e-5,
+                                                 table=rope, q_abs=q_abs, q_off=0, q_head_cols=d + rot, q_rot_off=d, halves=halves)
+        row(f"latent norm + rotated parts (halves) + cache write + query rows, {name}", f"the same with neighbouring pairs, {name}",
+            t_us(lambda: prep(True)), t_us(lambda: prep(False)),
+            nbytes=n * ((rank + rot + hq * rot) * 2 + (rank + rot) * 2 + hq * rank * 4 + hq * (rank + rot) * 4))
+        o_h = bf(hq, n, d)
+        gate = t_us(lambda: ops.heads_gate(o_h, proj, cols - hq * d))
+        row(f"heads back to token rows + sigmoid gate, {name}", f"the same kernel, {name}", gate, gate, nbytes=3 * n * hq * d * 2)
+        # ---- the experts
+        h = bf(n, width)
+        us_soft = _time_us(lambda: ops.moe_route(h, router, None, top=top, kind="softmax", padded=True), graph=True)
+        us_sig = _time_us(lambda: ops.moe_route(h, router, corr, top=top, n_groups=4, keep=2, padded=True), graph=True)
+        row(f"softmax router (logits, choice, weights, tiles), {name}", f"sigmoid router with groups, {name}", us_soft, us_sig,
+            nbytes=n * width * 2 + experts * width * 4)
+        routing = ops.moe_route(h, router, None, top=top, kind="softmax", padded=True)
+        used = len(set(routing.chosen.flatten().tolist()))
+        if ops.moe_small_takes(n, top, width, ffe, False):       # as the part chooses
+            mine = lambda: ops.moe_experts_small(h, routing, w_up, w_down, "relu2", gated=False, combine=False)
+            like = lambda: ops.moe_experts_small(h, routing, wgu, w_down)
+        else:
+            mine = lambda: ops.moe_experts_tc(h, routing, w_up, w_down, err, "relu2", gated=False, combine=False)
+            like = lambda: ops.moe_experts_tc(h, routing, wgu, w_down, err)
+        flops = 2.0 * n * top * ffe * width
+        kw = (dict(nbytes=2 * used * ffe * width * 2, like_bytes=3 * used * ffe * width * 2) if single else
+              dict(flops=2 * flops, like_flops=3 * flops))
+        row(f"ungated experts (up with relu squared, down), {name}", f"gated experts (gate, up, down, weighted sum), {name}",
+            t_us(mine), t_us(like), note=f"{used} of {experts} experts are read by the {n} tokens" if single else "", **kw)
+        # ---- the residual sum of both sublayers and the next norm
+        weighted, branch = mine(), bf(n, width)
+        if single:
+            from tokamak_b200.parts.base import linear
+            branch = linear(bf(n, hq * d), bf(width, hq * d) * 0.02, err=err)
+        ops.flush_chains()
+        normed = torch.empty(n, width, dtype=torch.bfloat16, device=dev)
+        b_bytes = branch.numel() * branch.element_size()
+        row(f"mixer + weighted sum of experts + residual + input norm, {name}", f"output norm + residual, {name}",
+            t_us(lambda: ops.sum_rmsnorm(resid, (branch, weighted), normed, w1, 1e-5)),
+            t_us(lambda: ops.branch_norm_add(resid, branch, w1, None, 1e-6, None, normed, 0.0)),
+            nbytes=n * width * (8 + 2 + top * weighted.y.element_size()) + b_bytes, like_bytes=n * width * (8 + 2) + b_bytes)
+        row(f"the same with the kept rows and a vector, {name}", f"output norm + residual, {name}",
+            t_us(lambda: ops.sum_rmsnorm(resid, (branch, weighted), normed, w1, 1e-5, extra=keep, vector=w1)),
+            t_us(lambda: ops.branch_norm_add(resid, branch, w1, None, 1e-6, None, normed, 0.0)),
+            nbytes=n * width * (12 + 2 + top * weighted.y.element_size()) + b_bytes, like_bytes=n * width * (8 + 2) + b_bytes)
+        if single:
+            logits = f32(n, vocab)
+            cap = t_us(lambda: ops.logits_scale_cap(logits, 1.0, 30.0))
+            row(f"logit cap, {name}", f"the same kernel, {name}", cap, cap, nbytes=2 * logits.numel() * 4)
+    assert err.tolist()[0] == 0, err.tolist()
+    return rows
+
+
 DESIGNS = {
     "ketalix": dict(name="Ketalix", config=ketalix_config, twin=("qwen3_twin", qwen3_twin), kernels=ketalix_kernels),
     "logivik": dict(name="Logivik", config=logivik_config, twin=("ketalix_twin", ketalix_config), kernels=logivik_kernels),
     "tarivik": dict(name="Tarivik", config=tarivik_config, twin=("ketalix_twin", ketalix_config), kernels=tarivik_kernels),
     "pukinex": dict(name="Pukinex", config=pukinex_config, twin=("ketalix_twin", ketalix_config), kernels=pukinex_kernels),
+    "puresun": dict(name="Puresun", config=puresun_config, twin=("logivik_latent_twin", logivik_latent_twin), kernels=puresun_kernels),
 }
 
 
@@ -1740,9 +1892,9 @@ def main() -> int:
     ap.add_argument("--sizes", default="8b", choices=["0.6b", "8b", "14b", "32b"],
                     help="layer sizes: of --workload (0.6b, 8b), or of the decode/prefill run (8b, the metric's "
                          "own, 14b, 32b)")
-    ap.add_argument("--design", default=None, choices=["ketalix", "logivik", "tarivik", "pukinex"],
+    ap.add_argument("--design", default=None, choices=sorted(DESIGNS),
                     help="measure another design instead: its prefill and decode throughput beside the engine's closest "
-                         "other model of equal layer sizes (Ketalix beside Qwen3, Logivik beside Ketalix), and its kernels "
+                         "other model of equal layer sizes (Ketalix beside Qwen3, Puresun beside Logivik, the rest beside Ketalix), and its kernels "
                          "alone beside their like kernels (--design-sizes)")
     ap.add_argument("--design-sizes", default="2b", choices=sorted(KETALIX_SIZES))
     ap.add_argument("--num-requests", type=int, default=32)

@@ -50,13 +50,14 @@ __device__ __forceinline__ void ld4_f32(const __nv_bfloat16* p, float (&v)[4]) {
   v[0] = __low2float(a); v[1] = __high2float(a); v[2] = __low2float(b); v[3] = __high2float(b);
 }
 
-constexpr int kMoeRouteWarps = 8;
+constexpr int kMoeRouteWarps = 8;             // warps of a block, and of one in a step of few tokens
+constexpr int kMoeRouteWarpsFew = 16;
 
 // h: [n_tokens, width] activation type; router: [experts, width] float32; one block per token.  Every warp
 // forms the logits of its share of the experts (a lane sums its elements in ascending order, the lanes are
 // added up by a butterfly: the same sum whatever else the step holds); the first warp makes the choice.
 template <typename T>
-__global__ void __launch_bounds__(kMoeRouteWarps * 32)
+__global__ void __launch_bounds__(kMoeRouteWarpsFew * 32)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
                  const float* __restrict__ correction, int* __restrict__ chosen,
                  float* __restrict__ weights, int n_tokens, int width, int experts, int n_groups,
@@ -72,11 +73,12 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
   const T* x = h + (size_t)t * width;
   const bool vec = (width & 3) == 0 && (reinterpret_cast<uintptr_t>(h) & (4 * sizeof(T) - 1)) == 0 &&
                    (reinterpret_cast<uintptr_t>(router) & 15) == 0;
-  for (int e = warp; e < experts; e += kMoeRouteWarps) {
+  for (int e = warp; e < experts; e += (int)(blockDim.x >> 5)) {
     const float* w = router + (size_t)e * width;
     float acc = 0.0f;
     if (vec) {
-      for (int i = lane * 4; i < width; i += 128) {
+#pragma unroll 8
+      for (int i = lane * 4; i < width; i += 128) {       // unrolled: the loads of several pieces are under way at a time
         float xv[4], wv[4];
         ld4_f32(x + i, xv); ld4_f32(w + i, wv);
         acc += xv[0] * wv[0]; acc += xv[1] * wv[1]; acc += xv[2] * wv[2]; acc += xv[3] * wv[3];
@@ -539,9 +541,10 @@ TK_API int tk_moe_route(const void* h, const float* router, const float* correct
     return (int)cudaErrorInvalidValue;
   }
   const size_t smem = (size_t)(2 * experts + n_groups) * sizeof(float);
+  const unsigned route_warps = n_tokens <= 148 && experts > tk::kMoeRouteWarps ? tk::kMoeRouteWarpsFew : tk::kMoeRouteWarps;
   cudaError_t e = cudaSuccess;
   TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::moe_route_kernel<T>, dim3((unsigned)n_tokens),
-                                             dim3(tk::kMoeRouteWarps * 32), smem, stream, (const T*)h, router, correction, chosen,
+                                             dim3(route_warps * 32), smem, stream, (const T*)h, router, correction, chosen,
                                              weights, n_tokens, width, experts, n_groups, keep, top, softmax));
   if (e != cudaSuccess) return (int)e;
   e = tk::launch(tk::moe_sort_kernel, dim3(1), dim3(1024), 0, stream, (const int*)chosen, order, tiles, n_tiles,
