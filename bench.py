@@ -1644,8 +1644,8 @@ def puresun_config(s: dict) -> dict:
          "mask": {"size": s["window"]}, "rot": {"base": 1e6, "dims": 64}}
     mlp = {"kind": "moe", "expert": {"ff": s["ff"] // PURESUN_TOP}, "router": {"experts": PURESUN_EXPERTS, "top": PURESUN_TOP}}
     layers = [{"type": "latent_attention", "mixer": m, "mlp": mlp} for _ in range(s["layers"] - 2)]
-    return {"architecture": "Puresun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
-            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+    return {"architecture": "Puresun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "logit_softcap": 50.0,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 7919, "mul_cur": 104729}},
             "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}
 
 
@@ -1702,7 +1702,7 @@ def puresun_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
         # ---- embedding
         resid, keep, last = torch.empty(n, width, device=dev), torch.empty(n, width, device=dev), torch.zeros(n_req, 1, dtype=torch.int32, device=dev)
         row(f"token rows + pair rows + the copy for the loop, {name}", f"token rows, {name}",
-            t_us(lambda: ops.embed_bigram(table_e, pairs, last, step, resid, mul_prev=31, mul_cur=17, keep=keep)),
+            t_us(lambda: ops.embed_bigram(table_e, pairs, last, step, resid, mul_prev=7919, mul_cur=104729, keep=keep)),
             t_us(lambda: ops.embed_gather(table_e, step.token_ids, resid, err)),
             nbytes=n * width * (2 + 2 + 4 + 4), like_bytes=n * width * (2 + 4))
         # ---- attention in the latent space

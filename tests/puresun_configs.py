@@ -54,8 +54,8 @@ PS_C = {
 }
 # head counts that fill no tile evenly, a single pass over a span that ends with the model
 PS_D = {
-    "architecture": "Puresun", "vocab": 222, "width": 192, "norm": {"eps": 1e-5}, "embedding": _bigram(31, 5, 3),
-    "loop": {"start": 1, "stop": 3, "times": 1}, "logit_softcap": 30.0,
+    "architecture": "Puresun", "vocab": 222, "width": 192, "norm": {"eps": 1e-5}, "embedding": _bigram(29, 5, 3),
+    "loop": {"start": 1, "stop": 3, "times": 1}, "logit_softcap": 25.0,
     "layers": [
         _layer(_mixer(18, 8, 16, 24, 80, 0.2, 20), _moe(72, 16, 1)),
         _layer(_mixer(7, 24, 16, 40, 48, 0.16, 100, base=2000.0), _moe(128, 5, 2)),

@@ -584,6 +584,24 @@ def test_greedy_generation_through_the_entry_point_float32(tag):
         assert o.output_token_ids == plain.greedy_generate(cfg, w, p, 10), len(p)
 
 
+def test_preemption_is_invisible_in_greedy_tokens_float32():
+    """A pool so small that requests are evicted and recomputed: the record of the previous token starts over with
+    the request, and the tokens are those of a large pool and of the plain implementation."""
+    from tokamak_b200 import LLM, SamplingParams
+    tag = "SC"                                   # windows of 33 and 80: the pool of the longer one runs out
+    folder = folder_of(tag, "float32")
+    prompts = [random_tokens(pc.ALL[tag][0]["vocab"], n, seed=3 * n) for n in (40, 55, 48, 60)]
+    params = SamplingParams(temperature=0.0, max_new_tokens=30)
+    got = {}
+    for pool in (1024, 192):
+        llm = LLM(folder, dtype="float32", block_size=8, max_seq_len=96, kv_pool_tokens=pool, max_batch_size=4)
+        got[pool] = [o.output_token_ids for o in llm.generate(prompt_token_ids=prompts, sampling_params=params)]
+        assert (llm.last_stats["preemptions"] > 0) == (pool == 192)
+    assert got[192] == got[1024]
+    cfg, w = plain.load_folder(folder)
+    assert got[1024][1] == plain.greedy_generate(cfg, w, prompts[1], 30)
+
+
 def test_greedy_generation_bfloat16_with_graphs_picks_top_tokens():
     """Decode steps replayed from CUDA graphs (every part of the design declares them safe): the tokens are
     those of the same engine with every step laid out by the host, and nearly the plain implementation's best
