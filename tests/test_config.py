@@ -73,8 +73,8 @@ def test_ignored_keys_and_window():
 
 
 def test_registry_errors():
-    assert supported_architectures() == ["Ketalix", "Logivik", "Pukinex", "Puresun", "Qwen3ForCausalLM", "Tarivik"]
-    with pytest.raises(ConfigError, match="Unsupported architecture 'LlamaForCausalLM'; supported: Ketalix, Logivik, Pukinex, Puresun, Qwen3ForCausalLM, Tarivik"):
+    assert supported_architectures() == ["Ketalix", "Logivik", "Pukinex", "Puresun", "Qwen3ForCausalLM", "Sofinex", "Tarivik"]
+    with pytest.raises(ConfigError, match="Unsupported architecture 'LlamaForCausalLM'; supported: Ketalix, Logivik, Pukinex, Puresun, Qwen3ForCausalLM, Sofinex, Tarivik"):
         architecture_of({"architectures": ["LlamaForCausalLM"]})
     with pytest.raises(ConfigError, match="<missing>"):
         architecture_of({})

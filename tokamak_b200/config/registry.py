@@ -152,3 +152,7 @@ def _load_builtin() -> None:
     if "Puresun" not in _ARCHITECTURES:
         from ..models import puresun
         register_architecture(Architecture(puresun.ARCHITECTURE, puresun.parse_config, puresun.model_spec))
+    if "Sofinex" not in _ARCHITECTURES:
+        from ..models import sofinex
+        register_architecture(Architecture(sofinex.ARCHITECTURE, sofinex.parse_config, sofinex.model_spec,
+                                           reads_tensor_shapes=True))

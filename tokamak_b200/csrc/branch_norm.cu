@@ -216,6 +216,134 @@ __global__ void __launch_bounds__(512) branch_norm_add_vec_kernel(float* __restr
   }
 }
 
+// Two branches that join together, each after a norm of its own:
+//   x = resid + a * rsqrt(mean(a^2) + eps_b) * w_a + b * rsqrt(mean(b^2) + eps_b) * w_b,   out = x * rsqrt(mean(x^2) + eps_n) * next_w
+struct BranchPairParams {
+  float* resid;
+  const void* branch[2];        // activation type, or null: float32 partial sums
+  const float* parts[2];
+  int n_parts[2];
+  size_t part_stride[2];
+  const float* post_w[2];
+  const float* next_w;
+  void* out;
+  const int* rows;
+  int hidden;
+  float eps_b, eps_n;
+};
+
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+  v.x = warp_sum(v.x); v.y = warp_sum(v.y);
+  __syncthreads();
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  const float2 r = lane < nwarps ? scratch[lane] : make_float2(0.0f, 0.0f);
+  return make_float2(warp_sum(r.x), warp_sum(r.y));
+}
+
+// Any width: both branches lie in shared memory, the first's place takes the new row.
+template <typename T>
+__global__ void branch_pair_norm_add_kernel(BranchPairParams p) {
+  extern __shared__ float row[];          // [2][hidden]
+  __shared__ float2 scratch[32];
+  pdl_trigger();
+  pdl_wait();
+  const int i = blockIdx.x, r = p.rows ? p.rows[i] : i, hidden = p.hidden;
+  float* x = p.resid + (size_t)r * hidden;
+  float2 ss = make_float2(0.0f, 0.0f);
+  for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+    float v[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      if (p.branch[j] != nullptr) {
+        v[j] = to_f32<T>(((const T*)p.branch[j])[(size_t)r * hidden + h]);
+      } else {
+        v[j] = 0.0f;
+        for (int s = 0; s < p.n_parts[j]; ++s) v[j] += p.parts[j][(size_t)s * p.part_stride[j] + (size_t)r * hidden + h];
+      }
+      row[j * hidden + h] = v[j];
+    }
+    ss.x += v[0] * v[0]; ss.y += v[1] * v[1];
+  }
+  ss = block_sum2(ss, scratch);
+  const float ra = rsqrtf(ss.x / (float)hidden + p.eps_b), rb = rsqrtf(ss.y / (float)hidden + p.eps_b);
+  float2 sx = make_float2(0.0f, 0.0f);
+  for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+    const float v = x[h] + (row[h] * ra * p.post_w[0][h] + row[hidden + h] * rb * p.post_w[1][h]);
+    if (p.rows == nullptr) x[h] = v;
+    row[h] = v;
+    sx.x += v * v;
+  }
+  const float rstd = rsqrtf(block_sum2(sx, scratch).x / (float)hidden + p.eps_n);
+  T* o = (T*)p.out + (size_t)i * hidden;
+  for (int h = threadIdx.x; h < hidden; h += blockDim.x) o[h] = from_f32<T>(row[h] * rstd * p.next_w[h]);
+}
+
+// Rows of a multiple of 4: everything stays in registers, the weights are asked for before the wait.
+template <typename T, int kChunks>
+__global__ void __launch_bounds__(512) branch_pair_norm_add_vec_kernel(BranchPairParams p) {
+  __shared__ float2 scratch[32];
+  pdl_trigger();
+  const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  const int hidden = p.hidden;
+  float4 wa[kChunks], wb[kChunks], nw[kChunks];
+#pragma unroll
+  for (int c = 0; c < kChunks; ++c) {
+    const int h = (threadIdx.x + c * blockDim.x) * 4;
+    wa[c] = wb[c] = nw[c] = zero;
+    if (h < hidden) { wa[c] = ld4<float>(p.post_w[0] + h); wb[c] = ld4<float>(p.post_w[1] + h); nw[c] = ld4<float>(p.next_w + h); }
+  }
+  pdl_wait();
+  const int i = blockIdx.x, r = p.rows ? p.rows[i] : i;
+  float* x = p.resid + (size_t)r * hidden;
+  float4 v[2][kChunks], xv[kChunks];
+  float2 ss = make_float2(0.0f, 0.0f);
+#pragma unroll
+  for (int c = 0; c < kChunks; ++c) {
+    const int h = (threadIdx.x + c * blockDim.x) * 4;
+    v[0][c] = v[1][c] = xv[c] = zero;
+    if (h >= hidden) continue;
+    xv[c] = ld4<float>(x + h);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      if (p.branch[j] != nullptr) {
+        v[j][c] = ld4<T>((const T*)p.branch[j] + (size_t)r * hidden + h);
+      } else {
+        const float* src = p.parts[j] + (size_t)r * hidden + h;
+        for (int s = 0; s < p.n_parts[j]; ++s) {
+          const float4 u = ld4<float>(src + (size_t)s * p.part_stride[j]);
+          v[j][c].x += u.x; v[j][c].y += u.y; v[j][c].z += u.z; v[j][c].w += u.w;
+        }
+      }
+    }
+    ss.x += v[0][c].x * v[0][c].x + v[0][c].y * v[0][c].y + v[0][c].z * v[0][c].z + v[0][c].w * v[0][c].w;
+    ss.y += v[1][c].x * v[1][c].x + v[1][c].y * v[1][c].y + v[1][c].z * v[1][c].z + v[1][c].w * v[1][c].w;
+  }
+  ss = block_sum2(ss, scratch);
+  const float ra = rsqrtf(ss.x / (float)hidden + p.eps_b), rb = rsqrtf(ss.y / (float)hidden + p.eps_b);
+  float2 sx = make_float2(0.0f, 0.0f);
+#pragma unroll
+  for (int c = 0; c < kChunks; ++c) {
+    const int h = (threadIdx.x + c * blockDim.x) * 4;
+    if (h >= hidden) continue;
+    xv[c].x += v[0][c].x * ra * wa[c].x + v[1][c].x * rb * wb[c].x;
+    xv[c].y += v[0][c].y * ra * wa[c].y + v[1][c].y * rb * wb[c].y;
+    xv[c].z += v[0][c].z * ra * wa[c].z + v[1][c].z * rb * wb[c].z;
+    xv[c].w += v[0][c].w * ra * wa[c].w + v[1][c].w * rb * wb[c].w;
+    if (p.rows == nullptr) st4<float>(x + h, xv[c]);
+    sx.x += xv[c].x * xv[c].x + xv[c].y * xv[c].y + xv[c].z * xv[c].z + xv[c].w * xv[c].w;
+  }
+  const float rstd = rsqrtf(block_sum2(sx, scratch).x / (float)hidden + p.eps_n);
+  T* o = (T*)p.out + (size_t)i * hidden;
+#pragma unroll
+  for (int c = 0; c < kChunks; ++c) {
+    const int h = (threadIdx.x + c * blockDim.x) * 4;
+    if (h < hidden) st4<T>(o + h, make_float4(xv[c].x * rstd * nw[c].x, xv[c].y * rstd * nw[c].y, xv[c].z * rstd * nw[c].z,
+                                              xv[c].w * rstd * nw[c].w));
+  }
+}
+
 }  // namespace tk
 
 TK_API int tk_branch_norm_add(float* resid, const void* branch, const float* parts, int n_parts,
@@ -274,5 +402,51 @@ TK_API int tk_branch_norm_add(float* resid, const void* branch, const float* par
                                    (size_t)hidden * sizeof(float), stream, resid, (const T*)branch, parts, n_parts,
                                    (size_t)part_stride, post_w, layer_scale, next_w, (T*)out, rows, hidden, eps_b,
                                    eps_n));
+  return (int)e;
+}
+
+TK_API int tk_branch_pair_norm_add(float* resid, const void* a, const float* a_parts, int a_n, long long a_stride,
+                                   const float* a_w, const void* b, const float* b_parts, int b_n, long long b_stride,
+                                   const float* b_w, const float* next_w, void* out, const int* rows, int n_rows,
+                                   int hidden, float eps_b, float eps_n, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (hidden < 1 || hidden > 12288 || (a == nullptr) == (a_parts == nullptr) || (b == nullptr) == (b_parts == nullptr) ||
+      a_w == nullptr || b_w == nullptr || next_w == nullptr || out == nullptr) {
+    return (int)cudaErrorInvalidValue;
+  }
+  tk::BranchPairParams p;
+  p.resid = resid; p.branch[0] = a; p.branch[1] = b; p.parts[0] = a_parts; p.parts[1] = b_parts;
+  p.n_parts[0] = a_n; p.n_parts[1] = b_n; p.part_stride[0] = (size_t)a_stride; p.part_stride[1] = (size_t)b_stride;
+  p.post_w[0] = a_w; p.post_w[1] = b_w; p.next_w = next_w; p.out = out; p.rows = rows; p.hidden = hidden;
+  p.eps_b = eps_b; p.eps_n = eps_n;
+  cudaError_t e = cudaSuccess;
+  if (hidden % 4 == 0 && hidden <= 8192) {
+    const int quads = hidden / 4;
+    const int threads = quads >= 512 ? 512 : (quads + 31) / 32 * 32;
+    const int chunks = (quads + threads - 1) / threads;
+#define TK_BRANCH_PAIR_VEC(K)                                                                                            \
+    TK_DISPATCH_DTYPE(dtype, T, (e = tk::launch(tk::branch_pair_norm_add_vec_kernel<T, K>, dim3((unsigned)n_rows),       \
+                                                dim3(threads), 0, stream, p)))
+    if (chunks <= 1) { TK_BRANCH_PAIR_VEC(1); }
+    else if (chunks <= 2) { TK_BRANCH_PAIR_VEC(2); }
+    else { TK_BRANCH_PAIR_VEC(4); }
+#undef TK_BRANCH_PAIR_VEC
+    return (int)e;
+  }
+  const size_t smem = (size_t)2 * hidden * sizeof(float);
+  const int threads = hidden >= 1024 ? 256 : 128;
+#define TK_BRANCH_PAIR(T)                                                                                              \
+  do {                                                                                                                 \
+    if (smem > 48 * 1024) {                                                                                            \
+      e = cudaFuncSetAttribute(tk::branch_pair_norm_add_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,        \
+                               (int)smem);                                                                             \
+      if (e != cudaSuccess) return (int)e;                                                                             \
+    }                                                                                                                  \
+    e = tk::launch(tk::branch_pair_norm_add_kernel<T>, dim3((unsigned)n_rows), dim3(threads), smem, stream, p);        \
+  } while (0)
+  if (dtype == tk::kF32) { TK_BRANCH_PAIR(float); }
+  else if (dtype == tk::kBF16) { TK_BRANCH_PAIR(__nv_bfloat16); }
+  else return (int)cudaErrorInvalidValue;
+#undef TK_BRANCH_PAIR
   return (int)e;
 }

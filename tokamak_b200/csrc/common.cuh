@@ -115,9 +115,10 @@ __device__ __forceinline__ float glu_act(float g, int act) {
   return g / (1.0f + expf(-g));
 }
 
-// Activations of an ungated unit: 0 = silu, 1 = the tanh form of gelu, 2 = relu(z)^2.
+// Activations of an ungated unit: 0 = silu, 1 = the tanh form of gelu, 2 = relu(z)^2, 3 = the exact gelu z Phi(z).
 __device__ __forceinline__ float unary_act(float z, int act) {
   if (act == 2) { const float r = fmaxf(z, 0.0f); return r * r; }
+  if (act == 3) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
   return glu_act(z, act);
 }
 

@@ -9,6 +9,9 @@
 // value head h reads q/k head h / (heads / kv_heads).  Per token and head, from two more columns,
 //   beta = sigmoid(b),    g = exp(-exp(A_log[h]) * softplus(a + dt_bias[h])).
 //
+// Or a decay per key channel: then a and dt_bias have one entry per head and key channel (a comes in rows of its own,
+// heads * key_dim wide), and g scales the rows of S:  S <- diag(g) S.
+//
 // A request's record in the state pool is  [ S: heads * key_dim * value_dim | tail: (K - 1) * channels ],
 // float32: the state and the last K - 1 inputs of the convolution (oldest first; zeros for a request
 // that has just begun).  Three kernels: delta_prepare_kernel (convolution, silu, unit norm, beta, g;
@@ -30,7 +33,8 @@ struct DeltaPrepareParams {
   int q_off, k_off, v_off, b_off, a_off;   // first columns of the pieces of a row
   const float* taps;          // [channels, n_taps]: q channels, k channels, v channels
   const float* a_log;         // [heads]
-  const float* dt_bias;       // [heads]
+  const float* dt_bias;       // [heads], or [heads, key_dim] with a decay per key channel
+  StackedInput a_in;          // channel decays: rows of heads * key_dim numbers a
   float* state;               // the pool of records
   long long rec_stride;       // floats per record
   long long tail_off;         // where the tail starts inside a record
@@ -41,7 +45,8 @@ struct DeltaPrepareParams {
   float* k_out;               // [n_tokens, kv_heads, key_dim]
   float* v_out;               // [n_tokens, heads, value_dim]
   float* beta_out;            // [n_tokens, heads]
-  float* g_out;               // [n_tokens, heads]
+  float* g_out;               // [n_tokens, heads], or [n_tokens, heads, key_dim]
+  int channel_decay;
   int* err;
   int n_tokens, n_reqs, n_slots, heads, kv_heads, dk, dv, n_taps;
   int move_tail;              // every request brings one token: the thread that reads a channel's tail also moves it on
@@ -137,6 +142,18 @@ __global__ void delta_prepare_kernel(DeltaPrepareParams p) {
     }
     const float f = rsqrtf(ss + p.unit_eps) * (kind == 0 ? p.q_scale : 1.0f);
     for (int e = lane; e < d; e += stride) dst[e] *= f;     // each thread rescales what it wrote itself
+  } else if (p.channel_decay) {
+    if (lane == 0) {
+      const float b = stacked_ld<T>(p.in, (size_t)t * p.in.row_stride + p.b_off + head);
+      p.beta_out[(size_t)t * p.heads + head] = 1.0f / (1.0f + expf(-b));
+    }
+    const float rate = -expf(p.a_log[head]);
+    const size_t row = (size_t)t * p.a_in.row_stride + (size_t)head * p.dk;
+    for (int e = lane; e < p.dk; e += stride) {
+      const float a = stacked_ld<T>(p.a_in, row + e) + p.dt_bias[(size_t)head * p.dk + e];
+      const float sp = a > 20.0f ? a : log1pf(expf(a));
+      p.g_out[((size_t)t * p.heads + head) * p.dk + e] = expf(rate * sp);
+    }
   } else if (lane == 0) {
     const size_t row = (size_t)t * p.in.row_stride;
     const float b = stacked_ld<T>(p.in, row + p.b_off + head);
@@ -181,14 +198,14 @@ __global__ void delta_tail_kernel(StackedInput in, int q_off, int k_off, int v_o
 }
 
 constexpr int kDeltaWarps = 8;
-constexpr int kDeltaBatch = 8;       // tokens staged in shared memory at a time (one per warp for the k.q products)
+constexpr int kDeltaBatch = 8;       // most tokens staged in shared memory at a time (one per warp for the k.q products)
 
 struct DeltaScanParams {
   const float* q;     // [n_tokens, kv_heads, dk]
   const float* k;
   const float* v;     // [n_tokens, heads, dv]
   const float* beta;  // [n_tokens, heads]
-  const float* g;
+  const float* g;     // [n_tokens, heads], or [n_tokens, heads, dk] with a decay per key channel
   float* state;       // records; S of head h at h * dk * dv, row-major [dk, dv]
   long long rec_stride;
   float* out;         // [n_tokens, heads, dv]
@@ -216,17 +233,20 @@ __device__ __forceinline__ void cp_async4(float* dst, const float* src) {
 // shuffles inside the warp (a fixed order), and since
 //   o = (g S + k u^T)^T q = (g S)^T q + u (k . q)
 // one meeting per token is enough.  No barrier stands between two tokens: the warps of a block only
-// share the staging of the inputs, which come in batches of kDeltaBatch tokens through shared memory,
-// the next batch on its way (cp.async) while this one is worked through.
-template <int kCP, int kRows>
+// share the staging of the inputs, which come in batches of kBatch tokens through shared memory,
+// the next batch on its way (cp.async) while this one is worked through.  kChannel: a decay per key channel,
+// staged like k (in smaller batches where the rows are long, for shared memory's sake).
+template <int kCP, int kRows, bool kChannel>
 __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanParams p) {
   constexpr int kGroups = 32 / kCP;                    // row groups of a warp
   constexpr int kRowsAll = kGroups * kRows;            // rows a warp can hold (>= dk)
   constexpr int kCols = kDeltaWarps * 2 * kCP;         // columns of a block
-  __shared__ __align__(16) float s_q[2][kDeltaBatch][kRowsAll];
-  __shared__ __align__(16) float s_k[2][kDeltaBatch][kRowsAll];
-  __shared__ __align__(8) float s_v[2][kDeltaBatch][kCols];
-  __shared__ float s_beta[2][kDeltaBatch], s_g[2][kDeltaBatch], s_kq[2][kDeltaBatch];
+  constexpr int kBatch = kChannel && kRowsAll > 128 ? kDeltaBatch / 2 : kDeltaBatch;
+  __shared__ __align__(16) float s_q[2][kBatch][kRowsAll];
+  __shared__ __align__(16) float s_k[2][kBatch][kRowsAll];
+  __shared__ __align__(16) float s_d[2][kBatch][kChannel ? kRowsAll : 4];     // channel decays
+  __shared__ __align__(8) float s_v[2][kBatch][kCols];
+  __shared__ float s_beta[2][kBatch], s_g[2][kBatch], s_kq[2][kBatch];
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -251,17 +271,19 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
     st[i].y = (ok1 && row_ok) ? S[(size_t)(row0 + i) * dv + 1] : 0.0f;
   }
   // rows beyond dk read q = k = 0 from shared memory and stay zero; so do columns beyond dv (v = 0)
-  for (int e = threadIdx.x; e < 2 * kDeltaBatch * kRowsAll; e += blockDim.x) {
+  for (int e = threadIdx.x; e < 2 * kBatch * kRowsAll; e += blockDim.x) {
     (&s_q[0][0][0])[e] = 0.0f;
     (&s_k[0][0][0])[e] = 0.0f;
+    if (kChannel) (&s_d[0][0][0])[e] = 0.0f;
   }
-  for (int e = threadIdx.x; e < 2 * kDeltaBatch * kCols; e += blockDim.x) (&s_v[0][0][0])[e] = 0.0f;
+  for (int e = threadIdx.x; e < 2 * kBatch * kCols; e += blockDim.x) (&s_v[0][0][0])[e] = 0.0f;
   __syncthreads();
 
   // q and k rows in 16-byte pieces where the rows allow it (key_dim a multiple of 4, the arrays aligned)
-  const bool vec = (dk & 3) == 0 && ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k)) & 15) == 0;
+  const bool vec = (dk & 3) == 0 && ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) |
+                                      (kChannel ? reinterpret_cast<uintptr_t>(p.g) : 0)) & 15) == 0;
   auto stage = [&](int b0, int buf) {
-    const int cnt = min(kDeltaBatch, n - b0);
+    const int cnt = min(kBatch, n - b0);
     if (vec) {
       const int quads = dk >> 2;
       for (int e = threadIdx.x; e < cnt * quads; e += blockDim.x) {
@@ -269,6 +291,7 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
         const size_t src = ((size_t)(t0 + b0 + i) * p.kv_heads + hk) * dk + x;
         cp_async16f(&s_q[buf][i][x], p.q + src);
         cp_async16f(&s_k[buf][i][x], p.k + src);
+        if (kChannel) cp_async16f(&s_d[buf][i][x], p.g + ((size_t)(t0 + b0 + i) * p.heads + h) * dk + x);
       }
     } else {
       for (int e = threadIdx.x; e < cnt * dk; e += blockDim.x) {
@@ -276,6 +299,7 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
         const size_t src = ((size_t)(t0 + b0 + i) * p.kv_heads + hk) * dk + x;
         cp_async4(&s_q[buf][i][x], p.q + src);
         cp_async4(&s_k[buf][i][x], p.k + src);
+        if (kChannel) cp_async4(&s_d[buf][i][x], p.g + ((size_t)(t0 + b0 + i) * p.heads + h) * dk + x);
       }
     }
     for (int e = threadIdx.x; e < cnt * kCols; e += blockDim.x) {
@@ -284,17 +308,17 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
     }
     if (threadIdx.x < cnt) {
       cp_async4(&s_beta[buf][threadIdx.x], p.beta + (size_t)(t0 + b0 + threadIdx.x) * p.heads + h);
-      cp_async4(&s_g[buf][threadIdx.x], p.g + (size_t)(t0 + b0 + threadIdx.x) * p.heads + h);
+      if (!kChannel) cp_async4(&s_g[buf][threadIdx.x], p.g + (size_t)(t0 + b0 + threadIdx.x) * p.heads + h);
     }
     asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
 
   if (n > 0) stage(0, 0);
-  for (int b0 = 0, buf = 0; b0 < n; b0 += kDeltaBatch, buf ^= 1) {
-    const int cnt = min(kDeltaBatch, n - b0);
+  for (int b0 = 0, buf = 0; b0 < n; b0 += kBatch, buf ^= 1) {
+    const int cnt = min(kBatch, n - b0);
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
     __syncthreads();          // this batch is there, and every warp has left the buffer that is staged next
-    if (b0 + kDeltaBatch < n) stage(b0 + kDeltaBatch, buf ^ 1);
+    if (b0 + kBatch < n) stage(b0 + kBatch, buf ^ 1);
     // k . q of every staged token: one warp a token, lanes over the rows, added in a fixed order
     if (warp < cnt) {
       float d = 0.0f;
@@ -305,10 +329,12 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
     __syncthreads();
     const float* kq_row = &s_k[buf][0][row0];
     const float* qq_row = &s_q[buf][0][row0];
+    const float* dq_row = &s_d[buf][0][kChannel ? row0 : 0];
     float* out_row = p.out + ((size_t)(t0 + b0) * p.heads + h) * dv + c0 + bcol;
 #pragma unroll 4
-    for (int i = 0; i < cnt; ++i, kq_row += kRowsAll, qq_row += kRowsAll, out_row += (size_t)p.heads * dv) {
-      const float gt = s_g[buf][i];
+    for (int i = 0; i < cnt; ++i, kq_row += kRowsAll, qq_row += kRowsAll, dq_row += kChannel ? kRowsAll : 0,
+                                 out_row += (size_t)p.heads * dv) {
+      const float gt = kChannel ? 0.0f : s_g[buf][i];
       const float2 g2 = make_float2(gt, gt);
       float2 kk[kRows];
       float2 a2 = make_float2(0.0f, 0.0f), b2 = a2, a3 = a2, b3 = a2;
@@ -318,8 +344,14 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
         const float4 q4 = *reinterpret_cast<const float4*>(qq_row + x);
         kk[x] = make_float2(k4.x, k4.x); kk[x + 1] = make_float2(k4.y, k4.y);
         kk[x + 2] = make_float2(k4.z, k4.z); kk[x + 3] = make_float2(k4.w, k4.w);
-        st[x] = mul2(st[x], g2); st[x + 1] = mul2(st[x + 1], g2);
-        st[x + 2] = mul2(st[x + 2], g2); st[x + 3] = mul2(st[x + 3], g2);
+        if (kChannel) {
+          const float4 d4 = *reinterpret_cast<const float4*>(dq_row + x);
+          st[x] = mul2(st[x], make_float2(d4.x, d4.x)); st[x + 1] = mul2(st[x + 1], make_float2(d4.y, d4.y));
+          st[x + 2] = mul2(st[x + 2], make_float2(d4.z, d4.z)); st[x + 3] = mul2(st[x + 3], make_float2(d4.w, d4.w));
+        } else {
+          st[x] = mul2(st[x], g2); st[x + 1] = mul2(st[x + 1], g2);
+          st[x + 2] = mul2(st[x + 2], g2); st[x + 3] = mul2(st[x + 3], g2);
+        }
         a2 = fma2(st[x], kk[x], a2); a3 = fma2(st[x + 1], kk[x + 1], a3);
         a2 = fma2(st[x + 2], kk[x + 2], a2); a3 = fma2(st[x + 3], kk[x + 3], a3);
         b2 = fma2(st[x], make_float2(q4.x, q4.x), b2); b3 = fma2(st[x + 1], make_float2(q4.y, q4.y), b3);
@@ -353,7 +385,90 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(DeltaScanP
   }
 }
 
+// The second half of low-rank projections in steps of few tokens: for each of two factors f,
+//   out[t, c] = sum_j a[t, off_f + j] * w_f[c, j]        (rank_f a multiple of 8; a rounded to T first, sums float32)
+// a are columns of a stacked projection (or of its partial sums).  Four lanes share an output channel (pieces of
+// eight factors in turn), a block takes 64 channels of one factor for kLowRankTokens tokens.
+constexpr int kLowRankTokens = 8;
+constexpr int kLowRankChannels = 64;
+
+struct LowRankParams {
+  StackedInput in;
+  const void* w[2];          // [channels, rank] T, 16-byte aligned
+  int off[2], rank[2], channels[2];
+  float* out[2];             // [n_tokens, channels]
+  int n_tokens, blocks0;     // blocks of the first factor
+};
+
+template <typename T> __device__ __forceinline__ void low_rank_ld8(const T* src, float (&v)[8]) {
+  const float4 a = ld4<T>(src), b = ld4<T>(src + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(4 * kLowRankChannels) low_rank_kernel(LowRankParams p) {
+  extern __shared__ __align__(16) float low_a[];       // [kLowRankTokens][rank]
+  pdl_trigger();
+  pdl_wait();
+  const int f = (int)blockIdx.x >= p.blocks0 ? 1 : 0;
+  const int rank = f ? p.rank[1] : p.rank[0], off = f ? p.off[1] : p.off[0], channels = f ? p.channels[1] : p.channels[0];
+  const int t0 = blockIdx.y * kLowRankTokens, cnt = min(kLowRankTokens, p.n_tokens - t0);
+  for (int e = threadIdx.x; e < kLowRankTokens * rank; e += blockDim.x) {
+    const int i = e / rank, j = e - i * rank;
+    low_a[e] = i < cnt ? to_f32<T>(from_f32<T>(stacked_ld<T>(p.in, (size_t)(t0 + i) * p.in.row_stride + off + j))) : 0.0f;
+  }
+  __syncthreads();
+  const int sub = threadIdx.x & 3;
+  const int c = (blockIdx.x - (f ? p.blocks0 : 0)) * kLowRankChannels + (threadIdx.x >> 2);
+  const bool live = c < channels;
+  float* out = f ? p.out[1] : p.out[0];
+  const T* w = (const T*)(f ? p.w[1] : p.w[0]) + (size_t)(live ? c : 0) * rank;
+  float acc[kLowRankTokens] = {};
+#pragma unroll 4
+  for (int j = sub * 8; j < rank; j += 32) {
+    float wv[8];
+    low_rank_ld8<T>(w + j, wv);
+#pragma unroll
+    for (int i = 0; i < kLowRankTokens; ++i) {
+      float av[8];
+      low_rank_ld8<float>(low_a + i * rank + j, av);
+#pragma unroll
+      for (int x = 0; x < 8; ++x) acc[i] += av[x] * wv[x];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kLowRankTokens; ++i) {
+    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 1);
+    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 2);
+    if (live && i < cnt && (i & 3) == sub) out[(size_t)(t0 + i) * channels + c] = acc[i];
+  }
+}
+
 }  // namespace tk
+
+TK_API int tk_low_rank(const void* x, const float* parts, int n_parts, long long part_stride, int row_stride, int off0,
+                       int rank0, const void* w0, int channels0, float* out0, int off1, int rank1, const void* w1,
+                       int channels1, float* out1, int n_tokens, int dtype, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  const int widest = rank0 > rank1 ? rank0 : rank1;
+  if ((x == nullptr) == (parts == nullptr) || rank0 < 8 || rank0 % 8 || channels0 < 1 || rank1 < 0 || rank1 % 8 ||
+      channels1 < 0 || (channels1 > 0 && rank1 < 8) || widest > 1024 || (((uintptr_t)w0 | (uintptr_t)w1) & 15)) {
+    return (int)cudaErrorInvalidValue;
+  }
+  tk::LowRankParams p;
+  p.in.x = x; p.in.parts = parts; p.in.n_parts = n_parts; p.in.row_stride = row_stride; p.in.part_stride = part_stride;
+  p.w[0] = w0; p.w[1] = w1; p.off[0] = off0; p.off[1] = off1; p.rank[0] = rank0; p.rank[1] = rank1;
+  p.channels[0] = channels0; p.channels[1] = channels1; p.out[0] = out0; p.out[1] = out1; p.n_tokens = n_tokens;
+  p.blocks0 = (channels0 + tk::kLowRankChannels - 1) / tk::kLowRankChannels;
+  const int blocks1 = (channels1 + tk::kLowRankChannels - 1) / tk::kLowRankChannels;
+  const long long tiles = ((long long)n_tokens + tk::kLowRankTokens - 1) / tk::kLowRankTokens;
+  if (tiles > 65535) return (int)cudaErrorInvalidValue;
+  const dim3 grid((unsigned)(p.blocks0 + blocks1), (unsigned)tiles);
+  cudaError_t e = cudaSuccess;
+  TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::low_rank_kernel<T>, grid, dim3(4 * tk::kLowRankChannels),
+                                             (size_t)tk::kLowRankTokens * widest * sizeof(float), stream, p));
+  return (int)e;
+}
 
 TK_API int tk_delta_prepare(const void* x, const float* parts, int n_parts, long long part_stride, int row_stride,
                             int q_off, int k_off, int v_off, int b_off, int a_off, const float* taps,
@@ -362,7 +477,9 @@ TK_API int tk_delta_prepare(const void* x, const float* parts, int n_parts, long
                             const int* req_slot, float* q_out, float* k_out, float* v_out, float* beta_out,
                             float* g_out, int* err, int n_tokens, int n_reqs, int n_slots, int heads, int kv_heads,
                             int dk, int dv, int n_taps, float unit_eps, float q_scale, int dtype, int move_tail_in_place,
-                            int shape, cudaStream_t stream) {
+                            int shape, const void* a_x, const float* a_parts, int a_n_parts, long long a_part_stride,
+                            int a_row_stride, cudaStream_t stream) {
+  // a_x or a_parts: rows [n_tokens, a_row_stride] of the channel decays' a (a_off is then not looked at)
   // move_tail_in_place: the caller vouches that every request brings at least one token, so that as many
   // tokens as requests means one token each; the kernel of the inputs then moves the tails on itself
   if (n_tokens <= 0 || n_reqs <= 0) return 0;
@@ -370,7 +487,11 @@ TK_API int tk_delta_prepare(const void* x, const float* parts, int n_parts, long
       n_taps < 1 || n_taps > tk::kDeltaMaxTaps || n_reqs > 65535) {
     return (int)cudaErrorInvalidValue;
   }
+  if (a_x != nullptr && a_parts != nullptr) return (int)cudaErrorInvalidValue;
   tk::DeltaPrepareParams p;
+  p.channel_decay = a_x != nullptr || a_parts != nullptr ? 1 : 0;
+  p.a_in.x = a_x; p.a_in.parts = a_parts; p.a_in.n_parts = a_n_parts; p.a_in.row_stride = a_row_stride;
+  p.a_in.part_stride = a_part_stride;
   p.in.x = x; p.in.parts = parts; p.in.n_parts = n_parts; p.in.row_stride = row_stride; p.in.part_stride = part_stride;
   p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.b_off = b_off; p.a_off = a_off;
   p.taps = taps; p.a_log = a_log; p.dt_bias = dt_bias; p.state = state; p.rec_stride = rec_stride; p.tail_off = tail_off;
@@ -412,7 +533,7 @@ TK_API int tk_delta_scan_cols(int heads, int dk, int dv) {
 TK_API int tk_delta_scan(const float* q, const float* k, const float* v, const float* beta, const float* g,
                          float* state, long long rec_stride, float* out, const int* req_q_start,
                          const int* req_q_len, const int* req_slot, int* err, int n_reqs, int n_slots, int heads,
-                         int kv_heads, int dk, int dv, int cols, cudaStream_t stream) {
+                         int kv_heads, int dk, int dv, int cols, int channel_decay, cudaStream_t stream) {
   if (n_reqs <= 0) return 0;
   if (cols <= 0) cols = tk_delta_scan_cols(heads, dk, dv);
   if (heads < 1 || kv_heads < 1 || heads % kv_heads || heads > 65535 || n_reqs > 65535 ||
@@ -431,7 +552,9 @@ TK_API int tk_delta_scan(const float* q, const float* k, const float* v, const f
   dim3 block(tk::kDeltaWarps * 32);
   cudaError_t e = cudaSuccess;
   // only the shapes that 256 key channels need are built
-#define TK_DELTA_LAUNCH(C, R) e = tk::launch(tk::delta_scan_kernel<C, R>, grid, block, 0, stream, p)
+#define TK_DELTA_LAUNCH(C, R)                                                                                 \
+  e = channel_decay ? tk::launch(tk::delta_scan_kernel<C, R, true>, grid, block, 0, stream, p)                \
+                    : tk::launch(tk::delta_scan_kernel<C, R, false>, grid, block, 0, stream, p)
   if (cp == 4) {
     if (rows <= 4) TK_DELTA_LAUNCH(4, 4); else if (rows <= 8) TK_DELTA_LAUNCH(4, 8);
     else if (rows <= 16) TK_DELTA_LAUNCH(4, 16); else TK_DELTA_LAUNCH(4, 32);

@@ -316,8 +316,8 @@ static int gemm_bf16_pair_launch(const void* x, const void* w, void* out, int* e
                                  long long ld_x, long long ld_w, long long ld_out, int mode, const int* tile_expert,
                                  int experts, cudaStream_t stream) {
   if (rows <= 0 || cols <= 0) return 0;
-  // modes 3, 4, 5: the plain product with an ungated activation (silu, gelu, relu squared) on its sums
-  const int unary = mode >= 3 && mode <= 5 ? mode - 2 : 0;
+  // modes 3 to 6: the plain product with an ungated activation (unary_act(sum, mode - 3)) on its sums
+  const int unary = mode >= 3 && mode <= 6 ? mode - 2 : 0;
   if (unary != 0) mode = 0;
   if (k <= 0 || k % 8 != 0 || ld_out % 8 != 0 || mode < 0 || mode > 2 || (mode != 0 && cols % 128 != 0) ||
       ((uintptr_t)out & 15u) != 0) {

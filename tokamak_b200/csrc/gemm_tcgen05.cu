@@ -599,8 +599,8 @@ static int launch_gemm(const void* r, const void* c, int rows, int cols, int k, 
 // of n_splits): that many consecutive splits form a thread-block cluster and store their sum.
 // epilogue = 1 (rows a multiple of 128 whose gate and up rows alternate in blocks of 64, all
 // splits in one cluster): out is bfloat16 [cols, rows / 2] = silu(gate) * up; epilogue = 4: the same with
-// the tanh form of gelu in silu's place.  epilogue = 5, 6, 7 (rows a multiple of 128, all splits in one cluster): out is
-// bfloat16 [cols, rows] = act(sum) with act = silu, the tanh form of gelu, relu squared.
+// the tanh form of gelu in silu's place.  epilogue = 5, 6, 7, 8 (rows a multiple of 128, all splits in one cluster): out is
+// bfloat16 [cols, rows] = act(sum) with act = silu, the tanh form of gelu, relu squared, the exact gelu.
 // epilogue = 2 (rows a multiple of 128, all splits in one cluster): nothing goes to out; the
 // sums are added to resid [cols, rows] (float32) in place, xb_out [cols, rows] receives
 // bf16(resid * norm_w) and sumsq_out [rows / 128, cols] the tiles' sums of squares of resid.
@@ -616,9 +616,9 @@ TK_API int tk_gemm_bf16_tcgen05(const void* r, const void* c, void* out, int* er
                                 float* sumsq_out, cudaStream_t stream) {
   const bool gelu = epilogue == tk::kGtEpiGeglu;
   if (gelu) epilogue = tk::kGtEpiSwiglu;
-  // epilogues 5, 6, 7: an ungated activation (silu, gelu, relu squared) on the sums of every row, stored as
+  // epilogues 5 to 8: an ungated activation (unary_act(sum, epilogue - 5)) on the sums of every row, stored as
   // bfloat16 [cols, rows]; they run as the gated epilogue with both halves of a tile as outputs
-  const int unary = epilogue >= 5 && epilogue <= 7 ? epilogue - 4 : 0;
+  const int unary = epilogue >= 5 && epilogue <= 8 ? epilogue - 4 : 0;
   if (unary != 0) epilogue = tk::kGtEpiSwiglu;
   if (epilogue < 0 || epilogue > tk::kGtEpiResidualNorm) return (int)cudaErrorInvalidValue;
   if (epilogue == tk::kGtEpiResidualNorm &&

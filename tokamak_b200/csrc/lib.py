@@ -19,7 +19,7 @@ _SIGNATURES: dict[str, list] = {
     "tk_embed_gather": [_P, c_int, _P, _P, c_int, c_int, c_int, c_float, c_int, _P, _P],
     "tk_embed_bigram": [_P, _P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_longlong, c_longlong, c_float, _P, _P],
-    "tk_sum_rmsnorm": [_P] + 2 * [_P, c_int, c_int, c_longlong, _P, _P] + [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float,
+    "tk_sum_rmsnorm": [_P] + 3 * [_P, c_int, c_int, c_longlong, _P, _P] + [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float,
                                                                           c_int, _P],
     "tk_step_begin": [_P, c_int, c_int, _P, c_int, _P, c_longlong, _P, _P, _P, _P, _P, c_int, c_int, _P, _P],
     "tk_decode_begin": [_P, c_int, c_int, _P, c_int, _P, c_longlong, _P, c_int, c_int, _P, _P, _P, _P, _P],
@@ -50,14 +50,18 @@ _SIGNATURES: dict[str, list] = {
     "tk_heads_gate": [_P, _P, _P, c_int, c_longlong, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P],
     "tk_delta_prepare": [_P, _P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P,
                          c_longlong, c_longlong, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P,
-                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, _P],
+                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int,
+                         _P, _P, c_int, c_longlong, c_int, _P],
+    "tk_low_rank": [_P, _P, c_int, c_longlong, c_int] + 2 * [c_int, c_int, _P, c_int, _P] + [c_int, c_int, _P],
     "tk_delta_scan": [_P, _P, _P, _P, _P, _P, c_longlong, _P, _P, _P, _P, _P,
-                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
     "tk_delta_scan_cols": [c_int, c_int, c_int],
     "tk_gemm_f32_batched": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong,
                             c_longlong, _P],
     "tk_branch_norm_add": [_P, _P, _P, c_int, c_longlong, _P, _P, _P, _P, _P, c_int, c_int, c_float, c_float,
                            c_int, c_int, c_int, _P],
+    "tk_branch_pair_norm_add": [_P] + 2 * [_P, _P, c_int, c_longlong, _P] + [_P, _P, _P, c_int, c_int, c_float, c_float, c_int,
+                                                                             _P],
     "tk_short_conv": [_P, _P, c_int, c_longlong, _P, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P, _P,
                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
     "tk_hgrn2_prepare": [_P, _P, c_int, c_longlong, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int,
@@ -75,7 +79,8 @@ _SIGNATURES: dict[str, list] = {
                              c_float, _P, c_int, c_int, c_int, c_int, c_int, _P],
     "tk_qkv_heads": [_P, _P, c_int, c_longlong, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_float,
                      _P, c_int, c_int, c_float, c_int, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P,
-                     c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+                     c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "tk_map_difference": [_P, _P, c_longlong, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, _P],
     "tk_hyper_mix_norm": [_P, _P, _P, c_int, c_longlong, c_int, _P, _P, _P, _P, _P, _P, _P, _P,
                           c_int, c_int, c_int, c_int, c_float, c_float, c_int, _P],
     "tk_logits_scale_cap": [_P, c_longlong, c_float, c_float, _P],
@@ -85,8 +90,7 @@ _SIGNATURES: dict[str, list] = {
                        c_float, c_int, _P],
     "tk_moe_tile_rows": [],
     "tk_moe_pad_rows": [],
-    "tk_moe_route": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                     _P],
+    "tk_moe_route": 11 * [_P] + 13 * [c_int] + [_P],
     "tk_moe_gather": [_P, c_longlong, _P, _P, c_int, c_int, c_int, _P],
     "tk_moe_combine_rows": [_P, _P, _P, _P, c_int, c_int, c_int, _P],
     "tk_moe_ffn": [_P, c_longlong, c_int, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P],
@@ -99,7 +103,7 @@ _SIGNATURES: dict[str, list] = {
     "tk_gla_prepare": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
                        c_float, c_float, c_int, _P],
     "tk_gla_scan": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
-    "tk_gla_out": [_P, _P, _P, c_int, c_int, c_int, _P, _P, c_int, c_float, c_int, c_int, c_int, c_float, c_int, _P],
+    "tk_gla_out": [_P, _P, _P, c_int, c_int, c_int, _P, _P, c_int, c_float, c_int, c_int, c_int, c_float, c_int, c_int, _P],
     "tk_attention_decode": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P,
                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_float, c_float, _P, c_int, _P, _P, c_int, _P],

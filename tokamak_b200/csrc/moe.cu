@@ -1,12 +1,18 @@
 // A mixture of feed-forward experts, gated or not, with a sigmoid or a softmax router.
 //
-//   s = sigmoid(W_r h), or s = W_r h for a softmax router         scores, float32
+//   s = sigmoid(W_r h), or s = W_r h for a softmax router over the chosen, or s = softmax(W_r h)      scores, float32
 //   c = s + correction                       choice scores
-//   the experts form equal groups of neighbours; a group's score is the sum of its two largest c; only
-//   experts of the `keep` best groups can be chosen; the `top` experts with the largest c are chosen
-//   g_e = s_e, or, for a softmax router, exp(s_e) / sum of exp(s) over the chosen experts only
+//   the experts form equal groups of neighbours; a group's score is the sum of its two largest c, or its
+//   largest; only experts of the `keep` best groups can be chosen; the `top` experts with the largest c are chosen
+//   g_e = s_e, or exp(s_e) / sum of exp(s) over the chosen experts only, or s_e / (sum of the chosen s + 1e-20)
 //   out = sum over the chosen e of g_e * W_down,e (act(W_gate,e h) * (W_up,e h))       gated experts
 //   out = sum over the chosen e of g_e * W_down,e act(W_up,e h)                        ungated ones
+//
+// The last outputs of the router may be identity experts, whose output is h itself: they take part in everything
+// up to the choice, then their weights are added up into one number per token (the pair itself is marked with
+// expert -1 and weight 0, and every reader skips such a pair).  A shared expert, which every token uses with the weight
+// sigmoid(z) of one more router row, is given as one or several experts behind the others (pieces of its inner
+// size, whose outputs add up) and takes the places behind a token's `top` choices.
 //
 // Five kernels.  moe_route_kernel: a block per token forms the logits, and its first warp makes the choice
 // (ties go to the lower index).  moe_sort_kernel: one block counts the (token, choice) pairs of every expert, lays the
@@ -53,28 +59,39 @@ __device__ __forceinline__ void ld4_f32(const __nv_bfloat16* p, float (&v)[4]) {
 constexpr int kMoeRouteWarps = 8;             // warps of a block, and of one in a step of few tokens
 constexpr int kMoeRouteWarpsFew = 16;
 
-// h: [n_tokens, width] activation type; router: [experts, width] float32; one block per token.  Every warp
-// forms the logits of its share of the experts (a lane sums its elements in ascending order, the lanes are
-// added up by a butterfly: the same sum whatever else the step holds); the first warp makes the choice.
+// One block per token.  Every warp forms the logits of its share of the router's rows (a lane sums its elements in
+// ascending order, the lanes are added up by a butterfly: the same sum whatever else the step holds); the first
+// warp makes the choice.
+enum MoeRouter : int { kRouteSigmoid = 0, kRouteSoftmaxChosen = 1, kRouteSoftmaxAll = 2 };
+
+struct MoeRouteParams {
+  const void* h;              // [n_tokens, width] activation type
+  const float* router;        // [outputs (+ 1 with a shared expert), width]
+  const float* correction;    // [outputs] or null
+  int* chosen;                // [n_tokens, top + shared]
+  float* weights;             // [n_tokens, top + shared]
+  float* identity_weight;     // [n_tokens] or null
+  int n_tokens, width, outputs, n_groups, keep, top, kind, group_best, normalize;
+  int identity;               // so many of the last outputs are identity experts
+  int shared;                 // pieces of the shared expert
+};
+
 template <typename T>
-__global__ void __launch_bounds__(kMoeRouteWarpsFew * 32)
-moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
-                 const float* __restrict__ correction, int* __restrict__ chosen,
-                 float* __restrict__ weights, int n_tokens, int width, int experts, int n_groups,
-                 int keep, int top, int softmax) {
+__global__ void __launch_bounds__(kMoeRouteWarpsFew * 32) moe_route_kernel(MoeRouteParams p) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x;
-  float* s = smem;
-  float* c = s + experts;
-  float* gs = c + experts;
-  const T* x = h + (size_t)t * width;
-  const bool vec = (width & 3) == 0 && (reinterpret_cast<uintptr_t>(h) & (4 * sizeof(T) - 1)) == 0 &&
-                   (reinterpret_cast<uintptr_t>(router) & 15) == 0;
-  for (int e = warp; e < experts; e += (int)(blockDim.x >> 5)) {
-    const float* w = router + (size_t)e * width;
+  const int outputs = p.outputs, width = p.width, n_groups = p.n_groups, rows = outputs + (p.shared > 0 ? 1 : 0);
+  float* s = smem;              // [outputs], and the shared expert's gate behind them
+  float* c = s + rows;
+  float* gs = c + outputs;
+  const T* x = (const T*)p.h + (size_t)t * width;
+  const bool vec = (width & 3) == 0 && (reinterpret_cast<uintptr_t>(p.h) & (4 * sizeof(T) - 1)) == 0 &&
+                   (reinterpret_cast<uintptr_t>(p.router) & 15) == 0;
+  for (int e = warp; e < rows; e += (int)(blockDim.x >> 5)) {
+    const float* w = p.router + (size_t)e * width;
     float acc = 0.0f;
     if (vec) {
 #pragma unroll 8
@@ -87,26 +104,32 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
       for (int i = lane; i < width; i += 32) acc += to_f32<T>(x[i]) * w[i];
     }
     acc = warp_sum(acc);
-    if (lane == 0) {
-      s[e] = softmax ? acc : 1.0f / (1.0f + expf(-acc));
-      c[e] = s[e] + (correction != nullptr ? correction[e] : 0.0f);
-    }
+    if (lane == 0) s[e] = e == outputs || p.kind == kRouteSigmoid ? 1.0f / (1.0f + expf(-acc)) : acc;
   }
   __syncthreads();
   if (warp != 0) return;
+  if (p.kind == kRouteSoftmaxAll) {
+    float m = -INFINITY, sum = 0.0f;
+    for (int e = lane; e < outputs; e += 32) m = fmaxf(m, s[e]);
+    m = warp_max(m);
+    for (int e = lane; e < outputs; e += 32) { const float v = expf(s[e] - m); s[e] = v; sum += v; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < outputs; e += 32) s[e] = s[e] / sum;
+  }
+  for (int e = lane; e < outputs; e += 32) c[e] = s[e] + (p.correction != nullptr ? p.correction[e] : 0.0f);
   __syncwarp();
-  const int size = experts / n_groups;
-  if (keep < n_groups) {
+  const int size = outputs / n_groups;
+  if (p.keep < n_groups) {
     for (int g = lane; g < n_groups; g += 32) {
       float a = -INFINITY, b = -INFINITY;          // the two largest
       for (int i = 0; i < size; ++i) {
         const float v = c[g * size + i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      gs[g] = size >= 2 ? a + b : a;
+      gs[g] = size >= 2 && !p.group_best ? a + b : a;
     }
     __syncwarp();
-    for (int it = 0; it < keep; ++it) {
+    for (int it = 0; it < p.keep; ++it) {
       float best = -INFINITY; int bi = 0x7fffffff;
       for (int g = lane; g < n_groups; g += 32) {
         const float v = gs[g];
@@ -116,33 +139,50 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
       if (lane == 0 && bi < n_groups) gs[bi] = INFINITY;      // taken
       __syncwarp();
     }
-    for (int e = lane; e < experts; e += 32) {
+    for (int e = lane; e < outputs; e += 32) {
       if (gs[e / size] != INFINITY) c[e] = -INFINITY;
     }
     __syncwarp();
   }
-  for (int it = 0; it < top; ++it) {
+  const int per = p.top + p.shared;
+  int* chosen = p.chosen + (size_t)t * per;
+  float* weights = p.weights + (size_t)t * per;
+  for (int it = 0; it < p.top; ++it) {
     float best = -INFINITY; int bi = 0x7fffffff;
-    for (int e = lane; e < experts; e += 32) {
+    for (int e = lane; e < outputs; e += 32) {
       const float v = c[e];
       if (v > best || (v == best && e < bi && v != -INFINITY)) { best = v; bi = e; }
     }
     warp_argmax(best, bi);
-    if (bi >= experts) bi = 0;        // fewer experts allowed than asked for: refused by the host
+    if (bi >= outputs) bi = 0;        // fewer experts allowed than asked for: refused by the host
     if (lane == 0) {
-      chosen[(size_t)t * top + it] = bi;
-      weights[(size_t)t * top + it] = s[bi];
+      chosen[it] = bi;
+      weights[it] = s[bi];
       c[bi] = -INFINITY;
     }
     __syncwarp();
   }
-  if (softmax && lane == 0) {       // the chosen experts' scores become weights that sum to one
-    float* w = weights + (size_t)t * top;
-    float m = w[0], sum = 0.0f;
-    for (int k = 1; k < top; ++k) m = fmaxf(m, w[k]);
-    for (int k = 0; k < top; ++k) { const float x = expf(w[k] - m); w[k] = x; sum += x; }
-    for (int k = 0; k < top; ++k) w[k] = w[k] / sum;
+  if (lane != 0) return;
+  if (p.kind == kRouteSoftmaxChosen) {       // the chosen experts' scores become weights that sum to one
+    float m = weights[0], sum = 0.0f;
+    for (int k = 1; k < p.top; ++k) m = fmaxf(m, weights[k]);
+    for (int k = 0; k < p.top; ++k) { const float v = expf(weights[k] - m); weights[k] = v; sum += v; }
+    for (int k = 0; k < p.top; ++k) weights[k] = weights[k] / sum;
   }
+  if (p.normalize) {
+    float sum = 1e-20f;
+    for (int k = 0; k < p.top; ++k) sum += weights[k];
+    for (int k = 0; k < p.top; ++k) weights[k] = weights[k] / sum;
+  }
+  const int experts = outputs - p.identity;
+  if (p.identity > 0) {
+    float own = 0.0f;
+    for (int k = 0; k < p.top; ++k) {
+      if (chosen[k] >= experts) { own += weights[k]; weights[k] = 0.0f; chosen[k] = -1; }
+    }
+    p.identity_weight[t] = own;
+  }
+  for (int k = 0; k < p.shared; ++k) { chosen[p.top + k] = experts + k; weights[p.top + k] = s[outputs]; }
 }
 
 // order: [pairs] the pairs (token * top + choice) expert by expert; tiles: [max_tiles, 3] (expert, first
@@ -151,7 +191,9 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router,
 // expert of every kMoePadRows-row tile of that layout, -1 for tiles that nobody uses.
 __global__ void moe_sort_kernel(const int* __restrict__ chosen, int* __restrict__ order, int* __restrict__ tiles,
                                 int* __restrict__ n_tiles, int pairs, int experts, int* __restrict__ pair_row,
-                                int* __restrict__ tile_expert, int max_pad_tiles) {
+                                int* __restrict__ tile_expert, int max_pad_tiles, int shared, int per) {
+  // the last `shared` of the experts are chosen by every token, in the last places of its `per` choices: their
+  // pairs are counted and placed by the token's number, without atomics
   __shared__ int count[kMoeMaxExperts], start[kMoeMaxExperts], cursor[kMoeMaxExperts], tile0[kMoeMaxExperts];
   __shared__ int pad0[kMoeMaxExperts];
   pdl_trigger();
@@ -160,8 +202,9 @@ __global__ void moe_sort_kernel(const int* __restrict__ chosen, int* __restrict_
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     const int e = chosen[i];
-    if (e >= 0 && e < experts) atomicAdd(&count[e], 1);
+    if (e >= 0 && e < experts - shared) atomicAdd(&count[e], 1);
   }
+  for (int e = experts - shared + (int)threadIdx.x; e < experts; e += blockDim.x) count[e] = pairs / per;
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0, tile = 0, pad = 0;
@@ -177,9 +220,11 @@ __global__ void moe_sort_kernel(const int* __restrict__ chosen, int* __restrict_
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     const int e = chosen[i];
     if (e >= 0 && e < experts) {
-      const int at = atomicAdd(&cursor[e], 1);
+      const int at = e < experts - shared ? atomicAdd(&cursor[e], 1) : i / per;
       order[start[e] + at] = i;
       if (pair_row != nullptr) pair_row[i] = pad0[e] * kMoePadRows + at;
+    } else if (pair_row != nullptr) {
+      pair_row[i] = -1;        // an identity expert: no row
     }
   }
   if (tile_expert != nullptr) {
@@ -285,7 +330,10 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
   if (idx >= (long long)n_tokens * width) return;
   const int t = (int)(idx / width), c = (int)(idx - (long long)t * width);
   float acc = 0.0f;
-  for (int k = 0; k < top; ++k) acc += weights[(size_t)t * top + k] * y[((size_t)t * top + k) * width + c];
+  for (int k = 0; k < top; ++k) {
+    const float w = weights[(size_t)t * top + k];
+    if (w != 0.0f) acc += w * y[((size_t)t * top + k) * width + c];        // a pair of weight 0 may have no row
+  }
   out[idx] = acc;
 }
 
@@ -297,6 +345,7 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ h, long long h_strid
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (long long)pairs * width16) return;
   const int pair = (int)(idx / width16), c = (int)(idx - (long long)pair * width16);
+  if (pair_row[pair] < 0) return;
   rows[(size_t)pair_row[pair] * width16 + c] = h[(size_t)(pair / top) * h_stride16 + c];
 }
 
@@ -313,7 +362,9 @@ __global__ void moe_combine_rows_kernel(const __nv_bfloat16* __restrict__ y, con
   float a0 = 0.0f, a1 = 0.0f;
   for (int k = 0; k < top; ++k) {
     const float w = weights[(size_t)t * top + k];
-    const float2 v = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(y + (size_t)pair_row[(size_t)t * top + k] * width)[c]);
+    if (w == 0.0f) continue;                       // a pair of weight 0 may have no row
+    const size_t pair = (size_t)t * top + k, row = pair_row != nullptr ? (size_t)pair_row[pair] : pair;
+    const float2 v = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(y + row * width)[c]);
     a0 += w * v.x; a1 += w * v.y;
   }
   reinterpret_cast<float2*>(out + (size_t)t * width)[c] = make_float2(a0, a1);
@@ -532,23 +583,30 @@ TK_API int tk_moe_tile_rows() { return tk::kMoeTileRows; }
 TK_API int tk_moe_pad_rows() { return tk::kMoePadRows; }
 
 TK_API int tk_moe_route(const void* h, const float* router, const float* correction, int* chosen, float* weights,
-                        int* order, int* tiles, int* n_tiles, int* pair_row, int* tile_expert, int max_pad_tiles,
-                        int n_tokens, int width, int experts, int n_groups, int keep, int top, int softmax, int dtype,
-                        cudaStream_t stream) {
+                        float* identity_weight, int* order, int* tiles, int* n_tiles, int* pair_row, int* tile_expert,
+                        int max_pad_tiles, int n_tokens, int width, int outputs, int n_groups, int keep, int top, int kind,
+                        int group_best, int normalize, int identity, int shared, int dtype, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (experts < 1 || experts > tk::kMoeMaxExperts || n_groups < 1 || experts % n_groups || keep < 1 || keep > n_groups ||
-      top < 1 || top > keep * (experts / n_groups)) {
+  const int experts = outputs - identity + shared;        // with matrices of their own
+  if (outputs < 1 || outputs > 4096 || experts < 1 || experts > tk::kMoeMaxExperts || n_groups < 1 ||
+      outputs % n_groups || keep < 1 || keep > n_groups || top < 1 || top > keep * (outputs / n_groups) || identity < 0 ||
+      identity > outputs || shared < 0 || (identity > 0 && identity_weight == nullptr) || kind < 0 || kind > 2) {
     return (int)cudaErrorInvalidValue;
   }
-  const size_t smem = (size_t)(2 * experts + n_groups) * sizeof(float);
-  const unsigned route_warps = n_tokens <= 148 && experts > tk::kMoeRouteWarps ? tk::kMoeRouteWarpsFew : tk::kMoeRouteWarps;
+  tk::MoeRouteParams p;
+  p.h = h; p.router = router; p.correction = correction; p.chosen = chosen; p.weights = weights;
+  p.identity_weight = identity_weight; p.n_tokens = n_tokens; p.width = width; p.outputs = outputs; p.n_groups = n_groups;
+  p.keep = keep; p.top = top; p.kind = kind; p.group_best = group_best; p.normalize = normalize; p.identity = identity;
+  p.shared = shared;
+  const size_t smem = (size_t)(2 * outputs + 1 + n_groups) * sizeof(float);
+  const unsigned route_warps = n_tokens <= 148 && outputs > tk::kMoeRouteWarps ? tk::kMoeRouteWarpsFew : tk::kMoeRouteWarps;
   cudaError_t e = cudaSuccess;
+  if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
   TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::moe_route_kernel<T>, dim3((unsigned)n_tokens),
-                                             dim3(route_warps * 32), smem, stream, (const T*)h, router, correction, chosen,
-                                             weights, n_tokens, width, experts, n_groups, keep, top, softmax));
+                                             dim3(route_warps * 32), smem, stream, p));
   if (e != cudaSuccess) return (int)e;
   e = tk::launch(tk::moe_sort_kernel, dim3(1), dim3(1024), 0, stream, (const int*)chosen, order, tiles, n_tiles,
-                 n_tokens * top, experts, pair_row, tile_expert, max_pad_tiles);
+                 n_tokens * (top + shared), experts, pair_row, tile_expert, max_pad_tiles, shared, top + shared);
   return (int)e;
 }
 

@@ -265,13 +265,13 @@ def add_rmsnorm(resid: torch.Tensor, delta: torch.Tensor | None, weight: torch.T
                                     float(eps), dtype_code(out.dtype), _stream()), "add_rmsnorm")
 
 
-SUM_NORM_TERMS = 2      # branches that one call of sum_rmsnorm adds
+SUM_NORM_TERMS = 3      # branches that one call of sum_rmsnorm adds
 
 
 def sum_rmsnorm(resid: torch.Tensor, terms, out: torch.Tensor, weight: torch.Tensor, eps: float, *,
                 rows: torch.Tensor | None = None, extra: torch.Tensor | None = None,
                 vector: torch.Tensor | None = None) -> None:
-    """``x = resid + terms[0] + terms[1] + extra + vector`` in float32 (written back unless ``rows`` selects rows), then
+    """``x = resid + terms[0] + terms[1] + terms[2] + extra + vector`` in float32 (written back unless ``rows`` selects rows), then
     ``out = weight * x * rsqrt(mean x^2 + eps)``.  A term (at most ``SUM_NORM_TERMS``) is a branch's output in the
     activation type, the float32 partial sums of a split product or :class:`WeightedRows`; ``extra`` is float32 rows
     like ``resid``, ``vector`` one float32 row that every token receives."""
@@ -596,6 +596,33 @@ def branch_norm_add(resid: torch.Tensor, branch: torch.Tensor | None, post_weigh
            "branch_norm_add")
 
 
+def branch_pair_norm_add(resid: torch.Tensor, a: torch.Tensor, a_weight: torch.Tensor, b: torch.Tensor,
+                         b_weight: torch.Tensor, branch_eps: float, next_weight: torch.Tensor, out: torch.Tensor,
+                         next_eps: float, rows: torch.Tensor | None = None) -> None:
+    """``x = resid + rmsnorm(a) * a_weight + rmsnorm(b) * b_weight`` (written back unless ``rows`` selects rows), ``out =
+    rmsnorm(x) * next_weight``; a branch is in the type of ``out`` or float32 partial sums ``[parts, tokens, hidden]``."""
+    _want(resid, torch.float32, "resid"); _want(out, None, "out")
+    n, hidden = resid.shape
+    args = []
+    for name, t, w in (("a", a, a_weight), ("b", b, b_weight)):
+        x, parts, n_parts, rows_t, width = _parts_of(t, out.dtype, name)
+        _want(w, torch.float32, name + "_weight")
+        if (rows_t, width) != (n, hidden) or w.numel() != hidden:
+            raise KernelError("a branch and the stream differ in shape")
+        args += [_ptr(x), _ptr(parts), n_parts, parts.stride(0) if parts is not None else 0, w.data_ptr()]
+    _want(next_weight, torch.float32, "next_weight")
+    if next_weight.numel() != hidden:
+        raise KernelError("next_weight does not match the width")
+    if rows is not None:
+        _want(rows, torch.int32, "rows")
+    n_rows = rows.numel() if rows is not None else n
+    if out.numel() < n_rows * hidden:
+        raise KernelError("out needs room for the rows")
+    _check(_lib().tk_branch_pair_norm_add(resid.data_ptr(), *args, next_weight.data_ptr(), out.data_ptr(), _ptr(rows),
+                                          n_rows, hidden, float(branch_eps), float(next_eps), dtype_code(out.dtype),
+                                          _stream()), "branch_pair_norm_add")
+
+
 def qkv_pairs(qkv: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
               positions: torch.Tensor, tok_req: torch.Tensor, req_slot: torch.Tensor, block_table: torch.Tensor,
               table: torch.Tensor | None, err: torch.Tensor, *, n_q_heads: int, n_kv_heads: int, rotary_dim: int,
@@ -708,9 +735,13 @@ def gla_scan(prep: torch.Tensor, state: torch.Tensor, req_q_start: torch.Tensor,
     return out
 
 
+GATES = {"silu": 0, "sigmoid": 1}
+
+
 def gla_out(o: torch.Tensor, proj: torch.Tensor | None, g_off: int, weight: torch.Tensor | None, eps: float,
-            dtype: torch.dtype, out: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
-    """``rmsnorm(o) * weight * silu(gate) * out_scale`` per (token, head) in the activation type
+            dtype: torch.dtype, out: torch.Tensor | None = None, out_scale: float = 1.0,
+            gate: str = "silu") -> torch.Tensor:
+    """``rmsnorm(o) * weight * act(gate) * out_scale`` (``gate``: ``silu`` or ``sigmoid``) per (token, head) in the activation type
     ``[tokens, heads * value_dim]``; the gate is read from ``proj`` at column ``g_off`` (``proj=None``: no gate);
     ``weight=None``: the heads are only divided by their root mean square.  ``out`` may be a column range of
     wider rows."""
@@ -732,8 +763,8 @@ def gla_out(o: torch.Tensor, proj: torch.Tensor | None, g_off: int, weight: torc
     if y.dtype != dtype or y.shape != (n, heads * dv) or y.stride(1) != 1:
         raise KernelError("out must be [tokens, heads * value_dim] in the activation type with dense rows")
     _check(_lib().tk_gla_out(o.data_ptr(), _ptr(x), _ptr(parts), n_parts, row, g_off, _ptr(weight), y.data_ptr(),
-                                y.stride(0), float(out_scale), n, heads, dv, float(eps), dtype_code(dtype), _stream()),
-           "gla_out")
+                                y.stride(0), float(out_scale), n, heads, dv, float(eps), GATES[gate], dtype_code(dtype),
+                                _stream()), "gla_out")
     return y
 
 
@@ -924,12 +955,12 @@ def qkv_rownorm(proj: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, 
                                     dtype_code(q_out.dtype), _stream()), "qkv_rownorm")
 
 
-UNARY_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
+UNARY_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "gelu": 3}
 
 
 def unary_act(x: torch.Tensor, dtype: torch.dtype, activation: str) -> torch.Tensor:
-    """``act(x)`` element by element in the activation type: ``silu``, ``gelu_tanh`` or ``relu2`` (the square of
-    relu).  ``x`` is ``[tokens, cols]`` in ``dtype`` or the float32 partial sums of a split product."""
+    """``act(x)`` element by element in the activation type: ``silu``, ``gelu_tanh``, ``relu2`` (the square of
+    relu) or ``gelu`` (exact, by the error function).  ``x`` is ``[tokens, cols]`` in ``dtype`` or the float32 partial sums of a split product."""
     if activation not in UNARY_ACTIVATIONS:
         raise KernelError(f"unknown activation {activation!r}; known: {', '.join(UNARY_ACTIVATIONS)}")
     xp, parts, n_parts, n, cols = _parts_of(x, dtype, "x")
@@ -1004,22 +1035,31 @@ def hyper_mix_norm(streams: torch.Tensor, branch: torch.Tensor | None, *, mix: t
 def qkv_heads(proj: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, step,
               block_table: torch.Tensor, *, q_off: int, k_off: int, v_off: int | None, q_bias=None, k_bias=None,
               v_bias=None, head_norm_eps: float | None = None, q_norm=None, k_norm=None, table=None,
-              rotary_dim: int = 0, halves: bool = False, temp_coef: float = 0.0, temp_every: int = 0) -> None:
+              rotary_dim: int = 0, halves: bool = False, temp_coef: float = 0.0, temp_every: int = 0,
+              norm_after: bool = False, maps: int = 1, k_dim: int | None = None, v_dim: int | None = None) -> None:
     """Queries, keys and values head by head from the columns of a stacked projection (activation type or
     float32 partial sums): biases, an RMS norm of every q and k head (``head_norm_eps``; ``q_norm`` / ``k_norm``: a
     weight of one head's size shared by all heads, or none), the query temperature
     ``1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)``, rotation over the first ``rotary_dim`` elements of the q
     and k heads by ``table`` (``[tokens, rotary_dim / 2, 2]`` float32; neighbouring pairs, or ``halves``); queries
     to ``q_out`` ``[tokens, Hq, d]``, keys and values into their pages.  ``v_off=None``: the values are the key
-    projection as it was before norm and rotation."""
-    n, hq, d = q_out.shape
-    num_pages, hkv, page_size, dk = k_cache.shape
-    dv = v_cache.shape[3]
-    if dk != d or not q_out.is_contiguous() or v_cache.shape[:3] != k_cache.shape[:3]:
+    projection as it was before norm and rotation.
+
+    ``norm_after``: the norm (and the temperature) follow the rotation.  ``maps``: the projection holds that many
+    pieces of ``k_dim`` elements per head, each normed and rotated on its own; a key row stores them one after the
+    other, every query piece has a row of its own (``Hq`` counts the pieces) with zeros outside its key piece's
+    place.  ``k_dim`` / ``v_dim``: sizes in the projection where the stored rows are longer (the rest is zero)."""
+    n, hq, k_row = q_out.shape
+    num_pages, hkv, page_size, stored_k = k_cache.shape
+    v_row = v_cache.shape[3]
+    d, dv = k_row // maps if k_dim is None else k_dim, v_row if v_dim is None else v_dim
+    if maps < 1 or hq % maps or maps * d > k_row or dv > v_row or (v_off is None and (maps != 1 or k_row != v_row)):
+        raise KernelError("qkv_heads: the pieces do not fit the stored rows")
+    if stored_k != k_row or not q_out.is_contiguous() or v_cache.shape[:3] != k_cache.shape[:3]:
         raise KernelError("qkv_heads shape mismatch")
     if max(d, dv) > 512:
         raise KernelError(f"head sizes {d} / {dv} are beyond the kernel's limit of 512")
-    for name, t, size in (("q_bias", q_bias, hq * d), ("k_bias", k_bias, hkv * d), ("v_bias", v_bias, hkv * dv),
+    for name, t, size in (("q_bias", q_bias, hq * d), ("k_bias", k_bias, hkv * maps * d), ("v_bias", v_bias, hkv * dv),
                           ("q_norm", q_norm, d), ("k_norm", k_norm, d)):
         if t is not None:
             _want(t, torch.float32, name)
@@ -1030,7 +1070,7 @@ def qkv_heads(proj: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_
         raise KernelError("proj and q_out differ in tokens")
     if v_off is None and dv != d:
         raise KernelError("values that are the keys have the keys' size")
-    spans = [(q_off, hq * d), (k_off, hkv * d)] + ([(v_off, hkv * dv)] if v_off is not None else [])
+    spans = [(q_off, hq * d), (k_off, hkv * maps * d)] + ([(v_off, hkv * dv)] if v_off is not None else [])
     if any(off < 0 or off + size > row for off, size in spans):
         raise KernelError("a column range lies outside the row")
     if table is not None:
@@ -1047,7 +1087,39 @@ def qkv_heads(proj: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_
                                   step.tok_req.data_ptr(), step.req_slot.data_ptr(), block_table.data_ptr(),
                                   step.req_q_len.data_ptr(), step.req_kv_len.data_ptr(), step.err.data_ptr(), n,
                                   step.req_slot.numel(), hq, hkv, d, dv, page_size, block_table.shape[1], num_pages,
-                                  dtype_code(q_out.dtype), _stream()), "qkv_heads")
+                                  int(bool(norm_after)), int(maps), k_row, v_row, dtype_code(q_out.dtype), _stream()),
+           "qkv_heads")
+
+
+ATTENTION_ROWS = (64, 128)      # row sizes of the tiled attention kernels
+
+
+def attention_row(size: int, dtype: torch.dtype) -> int:
+    """How many elements a head's stored key or value row of ``size`` gets so that the tiled attention kernels take
+    it: the next of their sizes (the rest is zero) in bfloat16, ``size`` itself where there is none."""
+    if dtype == torch.bfloat16:
+        for row in ATTENTION_ROWS:
+            if size <= row:
+                return row
+    return size
+
+
+def map_difference(a: torch.Tensor, v_dim: int, weight: float, eps: float, factor: float,
+                   out: torch.Tensor | None = None) -> torch.Tensor:
+    """Differential attention behind its two maps: ``o = a[:, 2h] - weight * a[:, 2h + 1]`` over the first ``v_dim``
+    elements of the rows ``a`` ``[tokens, 2 heads, row]``, divided by its root mean square (``eps`` inside the root) and
+    multiplied by ``factor``; ``[tokens, heads * v_dim]`` in the type of ``a``."""
+    _want(a, None, "a")
+    n, maps, row = a.shape
+    heads = maps // 2
+    if maps % 2 or not 1 <= v_dim <= min(row, 512):
+        raise KernelError("map_difference wants two maps per head and value sizes up to 512")
+    y = out if out is not None else torch.empty((n, heads * v_dim), dtype=a.dtype, device=a.device)
+    if y.dtype != a.dtype or y.shape != (n, heads * v_dim) or y.stride(1) != 1:
+        raise KernelError("out must be [tokens, heads * v_dim] in the type of the maps with dense rows")
+    _check(_lib().tk_map_difference(a.data_ptr(), y.data_ptr(), y.stride(0), n, heads, v_dim, row, float(weight),
+                                    float(eps), float(factor), dtype_code(a.dtype), _stream()), "map_difference")
+    return y
 
 
 def retention_prepare(proj: torch.Tensor, decay: torch.Tensor, table: torch.Tensor | None, *, dtype: torch.dtype,
@@ -1082,43 +1154,61 @@ def moe_tile_rows() -> int:
 
 
 class MoeRouting:
-    """What :func:`moe_route` leaves on the device: ``chosen`` / ``weights`` ``[tokens, top]``, the pairs
-    ``token * top + choice`` laid out expert by expert (``order``), and the products' row tiles.  With
+    """What :func:`moe_route` leaves on the device: ``chosen`` / ``weights`` ``[tokens, top + shared]``, the pairs
+    ``token * (top + shared) + choice`` laid out expert by expert (``order``), and the products' row tiles.  With
     ``padded``: also every pair's row in the layout whose experts start on whole tiles of
-    :func:`moe_pad_rows` rows (``pair_row``) and every such tile's expert (``tile_expert``, -1: unused)."""
+    :func:`moe_pad_rows` rows (``pair_row``) and every such tile's expert (``tile_expert``, -1: unused).  A pair of an
+    identity expert has the expert -1, the weight 0 and no row; ``identity_weight`` ``[tokens]`` is the sum of such
+    weights."""
 
-    def __init__(self, chosen, weights, order, tiles, n_tiles, max_tiles, pair_row=None, tile_expert=None):
+    def __init__(self, chosen, weights, order, tiles, n_tiles, max_tiles, pair_row=None, tile_expert=None,
+                 identity_weight=None):
         self.chosen, self.weights, self.order, self.tiles, self.n_tiles, self.max_tiles = (
             chosen, weights, order, tiles, n_tiles, max_tiles)
-        self.pair_row, self.tile_expert = pair_row, tile_expert
+        self.pair_row, self.tile_expert, self.identity_weight = pair_row, tile_expert, identity_weight
 
 
 def moe_pad_rows() -> int:
     return _lib().tk_moe_pad_rows()
 
 
-ROUTER_KINDS = {"sigmoid": 0, "softmax": 1}
+ROUTER_KINDS = {"sigmoid": 0, "softmax": 1, "softmax_all": 2}
+GROUP_SCORES = {"top2": 0, "best": 1}
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, *, top: int, n_groups: int = 1,
-              keep: int = 1, padded: bool = False, kind: str = "sigmoid") -> MoeRouting:
-    """Scores ``sigmoid(h router^T)`` in float32 (``kind="softmax"``: the logits themselves), choice by score plus
-    ``correction`` among the ``keep`` groups of neighbouring experts whose two best choice scores add up highest,
-    weights the plain scores (``softmax``: their softmax over the chosen experts only)."""
+              keep: int = 1, padded: bool = False, kind: str = "sigmoid", group_score: str = "top2",
+              normalize: bool = False, identity: int = 0, shared: int = 0) -> MoeRouting:
+    """Scores ``sigmoid(h router^T)`` in float32 (``kind="softmax"``: the logits themselves; ``"softmax_all"``: their
+    softmax), choice by score plus ``correction`` among the ``keep`` groups of neighbouring experts with the best
+    scores (``group_score``: the sum of the group's two best choice scores, or its best), weights the plain scores
+    (``softmax``: their softmax over the chosen experts only; ``normalize``: divided by their sum + 1e-20).
+
+    ``identity``: so many of the last outputs are identity experts (see :class:`MoeRouting`).  ``shared``: every token
+    also uses the experts ``outputs - identity`` and following, ``shared`` of them, with the weight sigmoid of the
+    router's last row, which is no output."""
     if kind not in ROUTER_KINDS:
         raise KernelError(f"unknown router {kind!r}; known: {', '.join(ROUTER_KINDS)}")
+    if group_score not in GROUP_SCORES:
+        raise KernelError(f"unknown group score {group_score!r}; known: {', '.join(GROUP_SCORES)}")
     _want(h, None, "h"); _want(router, torch.float32, "router")
     n, width = h.shape
-    experts = router.shape[0]
+    outputs = router.shape[0] - (1 if shared else 0)
+    experts = outputs - identity + shared
     if correction is not None:
         _want(correction, torch.float32, "correction")
-    if router.shape[1] != width or experts % n_groups or not 1 <= keep <= n_groups or not 1 <= top <= keep * (experts // n_groups):
+        if correction.numel() != outputs:
+            raise KernelError("one correction per router output is needed")
+    if (router.shape[1] != width or outputs < 1 or outputs % n_groups or not 1 <= keep <= n_groups
+            or not 1 <= top <= keep * (outputs // n_groups) or not 0 <= identity <= outputs or shared < 0 or experts < 1):
         raise KernelError("moe_route: sizes do not fit")
     dev = h.device
-    pairs = n * top
+    per = top + shared
+    pairs = n * per
     max_tiles = min(pairs, -(-pairs // moe_tile_rows()) + experts)
-    chosen = torch.empty((n, top), dtype=torch.int32, device=dev)
-    weights = torch.empty((n, top), dtype=torch.float32, device=dev)
+    chosen = torch.empty((n, per), dtype=torch.int32, device=dev)
+    weights = torch.empty((n, per), dtype=torch.float32, device=dev)
+    identity_weight = torch.empty((n, 1), dtype=torch.float32, device=dev) if identity else None
     order = torch.empty(pairs, dtype=torch.int32, device=dev)
     tiles = torch.empty((max_tiles, 3), dtype=torch.int32, device=dev)
     n_tiles = torch.empty(1, dtype=torch.int32, device=dev)
@@ -1127,10 +1217,11 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
         pair_row = torch.empty(pairs, dtype=torch.int32, device=dev)
         tile_expert = torch.empty(min(pairs, pairs // moe_pad_rows() + experts), dtype=torch.int32, device=dev)
     _check(_lib().tk_moe_route(h.data_ptr(), router.data_ptr(), _ptr(correction), chosen.data_ptr(), weights.data_ptr(),
-                                  order.data_ptr(), tiles.data_ptr(), n_tiles.data_ptr(), _ptr(pair_row), _ptr(tile_expert),
-                                  tile_expert.numel() if padded else 0, n, width, experts, n_groups,
-                                  keep, top, ROUTER_KINDS[kind], dtype_code(h.dtype), _stream()), "moe_route")
-    return MoeRouting(chosen, weights, order, tiles, n_tiles, max_tiles, pair_row, tile_expert)
+                               _ptr(identity_weight), order.data_ptr(), tiles.data_ptr(), n_tiles.data_ptr(),
+                               _ptr(pair_row), _ptr(tile_expert), tile_expert.numel() if padded else 0, n, width, outputs,
+                               n_groups, keep, top, ROUTER_KINDS[kind], GROUP_SCORES[group_score], int(bool(normalize)),
+                               int(identity), int(shared), dtype_code(h.dtype), _stream()), "moe_route")
+    return MoeRouting(chosen, weights, order, tiles, n_tiles, max_tiles, pair_row, tile_expert, identity_weight)
 
 
 MOE_SUMS, MOE_UNARY, MOE_GATED = 0, 1, 2        # what a product of the experts leaves (csrc/moe.cu)
@@ -1139,7 +1230,7 @@ MOE_SUMS, MOE_UNARY, MOE_GATED = 0, 1, 2        # what a product of the experts 
 @dataclass
 class WeightedRows:
     """The experts' outputs of a step before their weighted sum: token ``t``'s is the float32 sum over its
-    choices ``k`` of ``weights[t, k] * y[row(t, k)]``, with ``row`` the entry of ``pair_row`` or, without one, ``t *
+    choices ``k`` of ``weights[t, k] * y[row(t, k)]`` (choices of weight 0 are skipped and may have no row), with ``row`` the entry of ``pair_row`` or, without one, ``t *
     top + k``.  A kernel that reads it forms the sum itself (:func:`sum_rmsnorm`); :meth:`combine` is the sum."""
 
     y: torch.Tensor                     # [rows, width] bfloat16 or float32
@@ -1155,7 +1246,7 @@ class WeightedRows:
         top = self.weights.shape[1]
         out = torch.empty((n, width), dtype=torch.float32, device=self.y.device)
         if self.y.dtype == torch.bfloat16:
-            _check(_lib().tk_moe_combine_rows(self.y.data_ptr(), self.weights.data_ptr(), self.pair_row.data_ptr(),
+            _check(_lib().tk_moe_combine_rows(self.y.data_ptr(), self.weights.data_ptr(), _ptr(self.pair_row),
                                               out.data_ptr(), n, width, top, _stream()), "moe_combine_rows")
         else:
             _check(_lib().tk_moe_combine(self.y.data_ptr(), self.weights.data_ptr(), out.data_ptr(), n, width, top,
@@ -1751,7 +1842,7 @@ def delta_prepare(proj: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, d
                   records: torch.Tensor, tok_req: torch.Tensor, req_q_start: torch.Tensor, req_q_len: torch.Tensor,
                   req_slot: torch.Tensor, err: torch.Tensor, *, dtype: torch.dtype, q_off: int, k_off: int, v_off: int,
                   b_off: int, a_off: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, unit_eps: float,
-                  q_scale: float, shape: int = 0) -> tuple:
+                  q_scale: float, shape: int = 0, channel_a: torch.Tensor | None = None) -> tuple:
     """The float32 inputs of the delta-rule recurrence from the columns of the stacked projection
     ``proj`` (type ``dtype``, or float32 partial sums): short causal convolution (``taps`` float32
     ``[channels, K]``, channels in the order q, k, v) and silu on q, k and v, q and k heads scaled to
@@ -1759,6 +1850,8 @@ def delta_prepare(proj: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, d
     dt_bias))`` per head.  The convolution reads the inputs before the step from the tail of the
     requests' ``records`` (float32 ``[slots, floats]``, see :func:`delta_record_floats`) and moves the tail on
     (every request must bring at least one token: with as many tokens as requests the same kernel does both).
+    ``channel_a`` (``[N, heads * key_dim]`` like ``proj``: type ``dtype`` or float32 partial sums): a decay per head and key
+    channel from it instead of one per head; ``dt_bias`` is then ``[heads * key_dim]`` and ``g`` ``[N, H, dk]``.
     ``shape``: 0 lets the launcher choose a warp (many tokens) or a block (few) per head, 1 and 2 force one;
     the results are the same bits.
     Returns ``(q [N, Hk, dk], k [N, Hk, dk], v [N, H, dv], beta [N, H], g [N, H])``."""
@@ -1770,9 +1863,16 @@ def delta_prepare(proj: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, d
     floats, tail_off = delta_record_floats(heads, kv_heads, key_dim, value_dim, k_taps)
     if channels != 2 * hk + hv or records.dim() != 2 or records.shape[1] != floats:
         raise KernelError("taps must be [q + k + v channels, K] and the records sized by delta_record_floats")
-    if a_log.numel() != heads or dt_bias.numel() != heads:
-        raise KernelError("one A_log and one dt_bias per head are needed")
-    for off, size in ((q_off, hk), (k_off, hk), (v_off, hv), (b_off, heads), (a_off, heads)):
+    channel = channel_a is not None
+    if a_log.numel() != heads or dt_bias.numel() != heads * (key_dim if channel else 1):
+        raise KernelError("one A_log per head and one dt_bias per decay are needed")
+    a_args = (None, None, 0, 0, 0)
+    if channel:
+        ax, aparts, an, astride, n_a, a_row = _stacked(channel_a, dtype, "channel_a")
+        if (n_a, a_row) != (n, heads * key_dim):
+            raise KernelError("channel_a must be [tokens, heads * key_dim]")
+        a_args = (ax, aparts, an, astride, a_row)
+    for off, size in ((q_off, hk), (k_off, hk), (v_off, hv), (b_off, heads), (0 if channel else a_off, heads)):
         if off < 0 or off + size > row:
             raise KernelError("a column range lies outside the row")
     for name, t in (("tok_req", tok_req), ("req_q_start", req_q_start), ("req_q_len", req_q_len), ("req_slot", req_slot)):
@@ -1782,17 +1882,40 @@ def delta_prepare(proj: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, d
     k = torch.empty_like(q)
     v = torch.empty((n, heads, value_dim), dtype=torch.float32, device=dev)
     beta = torch.empty((n, heads), dtype=torch.float32, device=dev)
-    g = torch.empty_like(beta)
+    g = torch.empty((n, heads, key_dim) if channel else (n, heads), dtype=torch.float32, device=dev)
     _check(_lib().tk_delta_prepare(x, parts, n_parts, part_stride, row, q_off, k_off, v_off, b_off, a_off,
                                       taps.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), records.data_ptr(), floats,
                                       tail_off, tok_req.data_ptr(), req_q_start.data_ptr(), req_q_len.data_ptr(),
                                       req_slot.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
                                       g.data_ptr(), err.data_ptr(), n, req_slot.numel(), records.shape[0], heads,
                                       kv_heads, key_dim, value_dim, k_taps, float(unit_eps), float(q_scale),
-                                      dtype_code(dtype), 1, int(shape), _stream()), "delta_prepare")
+                                      dtype_code(dtype), 1, int(shape), *a_args, _stream()), "delta_prepare")
     global LAUNCHES
     LAUNCHES += 1 if k_taps > 1 and n != req_slot.numel() else 0       # the kernel that moves the tail on
     return q, k, v, beta, g
+
+
+LOW_RANK_MAX = 1024
+
+
+def low_rank(proj: torch.Tensor, dtype: torch.dtype, factors) -> list[torch.Tensor]:
+    """The second halves of one or two low-rank projections whose first halves are columns of ``proj`` (type ``dtype`` or
+    float32 partial sums): for every ``(offset, weight)`` of ``factors``, ``weight`` ``[channels, rank]`` with a rank in
+    whole eights, ``out = dtype(proj[:, offset:offset + rank]) @ weight^T`` as float32 ``[tokens, channels]``."""
+    x, parts, n_parts, part_stride, n, row = _stacked(proj, dtype, "proj")
+    if not 1 <= len(factors) <= 2:
+        raise KernelError("low_rank takes one factor or two")
+    args, outs = [], []
+    for off, w in factors:
+        _want(w, dtype, "weight")
+        channels, rank = w.shape
+        if off < 0 or off + rank > row or rank % 8 or not 8 <= rank <= LOW_RANK_MAX:
+            raise KernelError("a factor's columns lie outside the row, or its rank is not in whole eights up to 1024")
+        outs.append(torch.empty((n, channels), dtype=torch.float32, device=proj.device))
+        args += [off, rank, w.data_ptr(), channels, outs[-1].data_ptr()]
+    args += [0, 0, None, 0, None] * (2 - len(factors))
+    _check(_lib().tk_low_rank(x, parts, n_parts, part_stride, row, *args, n, dtype_code(dtype), _stream()), "low_rank")
+    return outs
 
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, g: torch.Tensor,
@@ -1800,13 +1923,15 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
                err: torch.Tensor, *, cols: int = 0) -> torch.Tensor:
     """The gated delta rule ``S = g S; u = beta (v - S^T k); S += k u^T; o = S^T q`` over every request's
     tokens of the step; the states ``[heads, dk, dv]`` lead the requests' float32 ``records`` and are
-    advanced in place.  Returns ``o`` float32 ``[tokens, heads, dv]``.  ``cols`` is the number of value
+    advanced in place.  ``g`` is ``[N, heads]``, or ``[N, heads, dk]`` with a decay per key channel (the rows of ``S``).
+    Returns ``o`` float32 ``[tokens, heads, dv]``.  ``cols`` is the number of value
     channels a block takes (64, 32 or 16: eight warps of 8, 4 or 2 columns; 0: what the sizes of the heads suggest)."""
     for name, t in (("q", q), ("k", k), ("v", v), ("beta", beta), ("g", g), ("records", records)):
         _want(t, torch.float32, name)
     n, kv_heads, dk = q.shape
     _, heads, dv = v.shape
-    if k.shape != q.shape or v.shape[0] != n or beta.shape != (n, heads) or g.shape != (n, heads) or heads % kv_heads:
+    if (k.shape != q.shape or v.shape[0] != n or beta.shape != (n, heads)
+            or g.shape not in ((n, heads), (n, heads, dk)) or heads % kv_heads):
         raise KernelError("the recurrence's inputs do not match one another")
     if records.dim() != 2 or records.shape[1] < heads * dk * dv:
         raise KernelError("a record is too short for the state")
@@ -1818,7 +1943,8 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
     _check(_lib().tk_delta_scan(q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), g.data_ptr(),
                                    records.data_ptr(), records.shape[1], out.data_ptr(), req_q_start.data_ptr(),
                                    req_q_len.data_ptr(), req_slot.data_ptr(), err.data_ptr(), req_slot.numel(),
-                                   records.shape[0], heads, kv_heads, dk, dv, int(cols), _stream()), "delta_scan")
+                                   records.shape[0], heads, kv_heads, dk, dv, int(cols), int(g.dim() == 3), _stream()),
+           "delta_scan")
     return out
 
 

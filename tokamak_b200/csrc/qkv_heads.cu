@@ -3,13 +3,21 @@
 //
 //   biases             z <- z + b                                   (q, k, v; each may be absent)
 //   head norm          x <- x / sqrt(mean_head(x^2) + eps) * w      (q and k; w of one head's size, shared by all
-//                                                                    heads, or absent: unit norm)
+//                                                                    heads, or absent: unit norm); before the
+//                                                                    rotation, or after it (norm_after)
 //   query temperature  q <- q * (1 + coef * ln(floor((p + 1) / every) + 1))   at position p
 //   rotation           over the first `rotary_dim` elements of every q and k head, either of neighbouring
 //                      pairs (2i, 2i + 1) or of halves (i, i + rotary_dim / 2); the pair (u, w) at angle a
 //                      becomes (u cos a - w sin a, w cos a + u sin a)
 //   values from keys   v = the key projection (with its bias) as it was before norm and rotation; the
 //                      projection then has no value columns
+//
+//   maps               a head's query and key are `maps` pieces of k_dim elements, each normed and rotated like a
+//                      head of its own.  The key row holds the pieces one after the other; every query piece
+//                      goes to a row of its own, at its key piece's place and with zeros elsewhere, so that its
+//                      product with the key row is the product of the two pieces
+//   stored rows        key (and query) rows of k_row >= maps * k_dim and value rows of v_row >= v_dim elements,
+//                      the rest zero (attention kernels that are built for a few row sizes)
 //
 // and the write of keys and values into their pages.  Everything is float32 and rounded once on store.
 // One warp per (token, head); a row of the input is a stacked projection (activation type or float32
@@ -28,17 +36,19 @@ struct QkvHeadsParams {
   const float* q_bias; const float* k_bias; const float* v_bias;
   const float* q_norm; const float* k_norm; // [k_dim] or null
   int head_norm;                            // 0: no norm
+  int norm_after;                           // the norm follows the rotation
   float eps;
   const float2* rope_table;                 // [n_tokens, rotary_dim / 2] (cos, sin) or null
   int rotary_dim, halves;
   float temp_coef; int temp_every;          // temp_every <= 0: no temperature
-  void* q_out;                              // [n_tokens, n_q_heads, k_dim]
-  void* k_cache;                            // [num_pages, n_kv_heads, page_size, k_dim]
-  void* v_cache;                            // [num_pages, n_kv_heads, page_size, v_dim]
+  void* q_out;                              // [n_tokens, n_q_heads, k_row]
+  void* k_cache;                            // [num_pages, n_kv_heads, page_size, k_row]
+  void* v_cache;                            // [num_pages, n_kv_heads, page_size, v_row]
   const int* positions; const int* tok_req; const int* req_slot; const int* block_table;
   const int* req_q_len; const int* req_kv_len;
   int* err;
   int n_tokens, n_reqs, n_q_heads, n_kv_heads, k_dim, v_dim, page_size, max_pages, num_pages;
+  int maps, k_row, v_row;                   // n_q_heads counts the pieces of the queries, n_kv_heads the key rows
 };
 
 template <typename T>
@@ -48,14 +58,15 @@ __global__ void qkv_heads_kernel(QkvHeadsParams p) {
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int own_v = p.v_off >= 0 ? p.n_kv_heads : 0;
-  const int heads_total = p.n_q_heads + p.n_kv_heads + own_v;
+  const int k_heads = p.n_kv_heads * p.maps;
+  const int heads_total = p.n_q_heads + k_heads + own_v;
   const int t = blockIdx.x;
   const int h = blockIdx.y * kHeadsWarps + warp;
   if (h >= heads_total) return;
   int kind, head;     // 0 = q, 1 = k, 2 = v
   if (h < p.n_q_heads) { kind = 0; head = h; }
-  else if (h < p.n_q_heads + p.n_kv_heads) { kind = 1; head = h - p.n_q_heads; }
-  else { kind = 2; head = h - p.n_q_heads - p.n_kv_heads; }
+  else if (h < p.n_q_heads + k_heads) { kind = 1; head = h - p.n_q_heads; }
+  else { kind = 2; head = h - p.n_q_heads - k_heads; }
   const int d = kind == 2 ? p.v_dim : p.k_dim;
   const int col = (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + head * d;
   const float* bias = kind == 0 ? p.q_bias : kind == 1 ? p.k_bias : p.v_bias;
@@ -66,8 +77,12 @@ __global__ void qkv_heads_kernel(QkvHeadsParams p) {
   T* dst = nullptr;
   T* dst_v = nullptr;          // values from keys: the same head of the value pages
   int zero_rows = 0;
+  // this warp's part of the stored row: [off, off + d), the row's rest behind the last piece, and all of a query's row
+  const int row_len = kind == 2 ? p.v_row : p.k_row;
+  const int piece = kind == 2 ? 0 : head % p.maps, off = piece * d;
+  const int tail = kind == 2 || piece == p.maps - 1 ? row_len - off : d;
   if (kind == 0) {
-    dst = (T*)p.q_out + ((size_t)t * p.n_q_heads + head) * d;
+    dst = (T*)p.q_out + ((size_t)t * p.n_q_heads + head) * row_len;
   } else {
     const int r = p.tok_req[t];
     if (r < 0 || r >= p.n_reqs) { if (lane == 0) set_error(p.err, kErrRequest, t, r, p.n_reqs); return; }
@@ -75,9 +90,9 @@ __global__ void qkv_heads_kernel(QkvHeadsParams p) {
     const int slot = pos - pidx * p.page_size;
     const int page = (pidx < p.max_pages) ? p.block_table[(size_t)p.req_slot[r] * p.max_pages + pidx] : -1;
     if (page < 0 || page >= p.num_pages) { if (lane == 0) set_error(p.err, kErrPage, t, pidx, page); return; }
-    const size_t row = ((size_t)page * p.n_kv_heads + head) * p.page_size + slot;
-    dst = (T*)(kind == 1 ? p.k_cache : p.v_cache) + row * d;
-    if (kind == 1 && p.v_off < 0) dst_v = (T*)p.v_cache + row * p.v_dim;
+    const size_t row = ((size_t)page * p.n_kv_heads + (kind == 1 ? head / p.maps : head)) * p.page_size + slot;
+    dst = (T*)(kind == 1 ? p.k_cache : p.v_cache) + row * row_len;
+    if (kind == 1 && p.v_off < 0) dst_v = (T*)p.v_cache + row * p.v_row;
     // the request's last token of this step clears the rest of a page that was begun in this step, so
     // that a live page never holds stale values behind the last position
     if (p.req_kv_len != nullptr) {
@@ -86,11 +101,21 @@ __global__ void qkv_heads_kernel(QkvHeadsParams p) {
     }
   }
   for (int z = 1; z <= zero_rows; ++z) {
-    for (int e = lane; e < d; e += 32) {
-      dst[(size_t)z * d + e] = from_f32<T>(0.0f);
-      if (dst_v != nullptr) dst_v[(size_t)z * d + e] = from_f32<T>(0.0f);
+    for (int e = lane; e < tail; e += 32) {
+      dst[(size_t)z * row_len + off + e] = from_f32<T>(0.0f);
+      if (dst_v != nullptr) dst_v[(size_t)z * row_len + e] = from_f32<T>(0.0f);
     }
   }
+  if (kind == 0) {
+    for (int e = lane; e < off; e += 32) dst[e] = from_f32<T>(0.0f);
+    for (int e = off + d + lane; e < row_len; e += 32) dst[e] = from_f32<T>(0.0f);
+  } else {
+    for (int e = d + lane; e < tail; e += 32) {
+      dst[off + e] = from_f32<T>(0.0f);
+      if (dst_v != nullptr) dst_v[e] = from_f32<T>(0.0f);
+    }
+  }
+  dst += off;
 
   float* x = s_head[warp];
   float ss = 0.0f;
@@ -102,16 +127,23 @@ __global__ void qkv_heads_kernel(QkvHeadsParams p) {
     if (dst_v != nullptr) dst_v[e] = from_f32<T>(v);
   }
   if (kind == 2) return;
-  float factor = 1.0f;
-  if (p.head_norm) factor = rsqrtf(warp_sum(ss) / (float)d + p.eps);
+  float factor = 1.0f, last = 1.0f;        // in front of the rotation, behind it
+  if (p.head_norm && !p.norm_after) factor = rsqrtf(warp_sum(ss) / (float)d + p.eps);
   if (kind == 0 && p.temp_every > 0) {
-    factor *= 1.0f + p.temp_coef * logf(floorf((float)(pos + 1) / (float)p.temp_every) + 1.0f);
+    (p.norm_after ? last : factor) *= 1.0f + p.temp_coef * logf(floorf((float)(pos + 1) / (float)p.temp_every) + 1.0f);
   }
-  const float* w = p.head_norm ? (kind == 0 ? p.q_norm : p.k_norm) : nullptr;
+  const float* w_norm = p.head_norm ? (kind == 0 ? p.q_norm : p.k_norm) : nullptr;
+  const float* w = p.norm_after ? nullptr : w_norm;
   __syncwarp();
   const int r = p.rope_table != nullptr ? p.rotary_dim : 0, half = r >> 1;
   const float2* tab = p.rope_table + (size_t)t * half;
-  for (int e = lane; e < d; e += 32) {
+  float kept[kHeadsMaxDim / 32];
+  float ss_after = 0.0f;
+#pragma unroll
+  for (int k = 0; k < kHeadsMaxDim / 32; ++k) {
+    const int e = lane + 32 * k;
+    kept[k] = 0.0f;
+    if (e >= d) continue;
     float v = x[e] * factor * (w != nullptr ? w[e] : 1.0f);
     if (e < r) {
       int partner, idx; bool first;
@@ -121,7 +153,16 @@ __global__ void qkv_heads_kernel(QkvHeadsParams p) {
       const float2 cs = tab[idx];
       v = first ? v * cs.x - o * cs.y : v * cs.x + o * cs.y;
     }
-    dst[e] = from_f32<T>(v);
+    if (!p.norm_after) { dst[e] = from_f32<T>(v); continue; }
+    kept[k] = v;
+    ss_after += v * v;
+  }
+  if (!p.norm_after) return;
+  if (p.head_norm) last *= rsqrtf(warp_sum(ss_after) / (float)d + p.eps);
+#pragma unroll
+  for (int k = 0; k < kHeadsMaxDim / 32; ++k) {
+    const int e = lane + 32 * k;
+    if (e < d) dst[e] = from_f32<T>(kept[k] * last * (w_norm != nullptr ? w_norm[e] : 1.0f));
   }
 }
 
@@ -135,14 +176,15 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int own_v = p.v_off >= 0 ? p.n_kv_heads : 0;
-  const int heads_total = p.n_q_heads + p.n_kv_heads + own_v;
+  const int k_heads = p.n_kv_heads * p.maps;
+  const int heads_total = p.n_q_heads + k_heads + own_v;
   const int t = blockIdx.x;
   const int h = blockIdx.y * kHeadsWarps + warp;
   if (h >= heads_total) return;
   int kind, head;     // 0 = q, 1 = k, 2 = v
   if (h < p.n_q_heads) { kind = 0; head = h; }
-  else if (h < p.n_q_heads + p.n_kv_heads) { kind = 1; head = h - p.n_q_heads; }
-  else { kind = 2; head = h - p.n_q_heads - p.n_kv_heads; }
+  else if (h < p.n_q_heads + k_heads) { kind = 1; head = h - p.n_q_heads; }
+  else { kind = 2; head = h - p.n_q_heads - k_heads; }
   const int d = kind == 2 ? p.v_dim : p.k_dim;
   const int col = (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + head * d;
   const float* bias = kind == 0 ? p.q_bias : kind == 1 ? p.k_bias : p.v_bias;
@@ -153,8 +195,12 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
   T* dst = nullptr;
   T* dst_v = nullptr;
   int zero_rows = 0;
+  // this warp's part of the stored row: [off, off + d), the row's rest behind the last piece, and all of a query's row
+  const int row_len = kind == 2 ? p.v_row : p.k_row;
+  const int piece = kind == 2 ? 0 : head % p.maps, off = piece * d;
+  const int tail = kind == 2 || piece == p.maps - 1 ? row_len - off : d;
   if (kind == 0) {
-    dst = (T*)p.q_out + ((size_t)t * p.n_q_heads + head) * d;
+    dst = (T*)p.q_out + ((size_t)t * p.n_q_heads + head) * row_len;
   } else {
     const int r = p.tok_req[t];
     if (r < 0 || r >= p.n_reqs) { if (lane == 0) set_error(p.err, kErrRequest, t, r, p.n_reqs); return; }
@@ -162,9 +208,9 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
     const int slot = pos - pidx * p.page_size;
     const int page = (pidx < p.max_pages) ? p.block_table[(size_t)p.req_slot[r] * p.max_pages + pidx] : -1;
     if (page < 0 || page >= p.num_pages) { if (lane == 0) set_error(p.err, kErrPage, t, pidx, page); return; }
-    const size_t row = ((size_t)page * p.n_kv_heads + head) * p.page_size + slot;
-    dst = (T*)(kind == 1 ? p.k_cache : p.v_cache) + row * d;
-    if (kind == 1 && p.v_off < 0) dst_v = (T*)p.v_cache + row * p.v_dim;
+    const size_t row = ((size_t)page * p.n_kv_heads + (kind == 1 ? head / p.maps : head)) * p.page_size + slot;
+    dst = (T*)(kind == 1 ? p.k_cache : p.v_cache) + row * row_len;
+    if (kind == 1 && p.v_off < 0) dst_v = (T*)p.v_cache + row * p.v_row;
     if (p.req_kv_len != nullptr) {
       const int kv_len = p.req_kv_len[r], q_len = p.req_q_len[r];
       if (pos == kv_len - 1 && pos - slot >= kv_len - q_len) zero_rows = p.page_size - 1 - slot;
@@ -173,11 +219,22 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
   const int chunks = d >> 2;
   const float4 zero4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   for (int z = 1; z <= zero_rows; ++z) {
-    for (int i = lane; i < chunks; i += 32) {
-      st4<T>(dst + (size_t)z * d + 4 * i, zero4);
-      if (dst_v != nullptr) st4<T>(dst_v + (size_t)z * d + 4 * i, zero4);
+    for (int i = lane; i < tail >> 2; i += 32) {
+      st4<T>(dst + (size_t)z * row_len + off + 4 * i, zero4);
+      if (dst_v != nullptr) st4<T>(dst_v + (size_t)z * row_len + 4 * i, zero4);
     }
   }
+  if (kind == 0) {
+    for (int e = 4 * lane; e < row_len; e += 128) {
+      if (e < off || e >= off + d) st4<T>(dst + e, zero4);
+    }
+  } else {
+    for (int e = d + 4 * lane; e < tail; e += 128) {
+      st4<T>(dst + off + e, zero4);
+      if (dst_v != nullptr) st4<T>(dst_v + e, zero4);
+    }
+  }
+  dst += off;
 
   float* x = s_head[warp];
   float4 own[4];
@@ -199,15 +256,17 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
     if (dst_v != nullptr) st4<T>(dst_v + 4 * i, v);
   }
   if (kind == 2) return;
-  float factor = 1.0f;
-  if (p.head_norm) factor = rsqrtf(warp_sum(ss) / (float)d + p.eps);
+  float factor = 1.0f, last = 1.0f;        // in front of the rotation, behind it
+  if (p.head_norm && !p.norm_after) factor = rsqrtf(warp_sum(ss) / (float)d + p.eps);
   if (kind == 0 && p.temp_every > 0) {
-    factor *= 1.0f + p.temp_coef * logf(floorf((float)(pos + 1) / (float)p.temp_every) + 1.0f);
+    (p.norm_after ? last : factor) *= 1.0f + p.temp_coef * logf(floorf((float)(pos + 1) / (float)p.temp_every) + 1.0f);
   }
-  const float* w = p.head_norm ? (kind == 0 ? p.q_norm : p.k_norm) : nullptr;
+  const float* w_norm = p.head_norm ? (kind == 0 ? p.q_norm : p.k_norm) : nullptr;
+  const float* w = p.norm_after ? nullptr : w_norm;
   __syncwarp();
   const int r = p.rope_table != nullptr ? p.rotary_dim : 0, half = r >> 1;
   const float2* tab = p.rope_table + (size_t)t * half;
+  float ss_after = 0.0f;
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const int i = lane + 32 * k;
@@ -228,7 +287,22 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
         }
       }
     }
-    st4<T>(dst + 4 * i, make_float4(v[0], v[1], v[2], v[3]));
+    own[k] = make_float4(v[0], v[1], v[2], v[3]);
+    if (!p.norm_after) st4<T>(dst + 4 * i, own[k]);
+    ss_after += v[0] * v[0]; ss_after += v[1] * v[1]; ss_after += v[2] * v[2]; ss_after += v[3] * v[3];
+  }
+  if (!p.norm_after) return;
+  if (p.head_norm) last *= rsqrtf(warp_sum(ss_after) / (float)d + p.eps);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int i = lane + 32 * k;
+    if (i >= chunks) continue;
+    float4 v = make_float4(own[k].x * last, own[k].y * last, own[k].z * last, own[k].w * last);
+    if (w_norm != nullptr) {
+      const float4 w4 = *reinterpret_cast<const float4*>(w_norm + 4 * i);
+      v.x *= w4.x; v.y *= w4.y; v.z *= w4.z; v.w *= w4.w;
+    }
+    st4<T>(dst + 4 * i, v);
   }
 }
 
@@ -241,8 +315,13 @@ TK_API int tk_qkv_heads(const void* x, const float* parts, int n_parts, long lon
                         void* q_out, void* k_cache, void* v_cache, const int* positions, const int* tok_req,
                         const int* req_slot, const int* block_table, const int* req_q_len, const int* req_kv_len,
                         int* err, int n_tokens, int n_reqs, int n_q_heads, int n_kv_heads, int k_dim, int v_dim,
-                        int page_size, int max_pages, int num_pages, int dtype, cudaStream_t stream) {
+                        int page_size, int max_pages, int num_pages, int norm_after, int maps, int k_row, int v_row,
+                        int dtype, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
+  if (maps < 1 || n_q_heads % maps || k_row < maps * k_dim || v_row < v_dim ||
+      (v_off < 0 && (maps != 1 || k_row != v_row))) {
+    return (int)cudaErrorInvalidValue;
+  }
   if ((x == nullptr) == (parts == nullptr) || n_q_heads < 1 || n_kv_heads < 1 || k_dim < 1 || v_dim < 1 ||
       k_dim > tk::kHeadsMaxDim || v_dim > tk::kHeadsMaxDim || rotary_dim < 0 || rotary_dim > k_dim ||
       (rotary_dim & 1) || (v_off < 0 && v_dim != k_dim)) {
@@ -259,10 +338,11 @@ TK_API int tk_qkv_heads(const void* x, const float* parts, int n_parts, long lon
   p.req_q_len = req_q_len; p.req_kv_len = req_kv_len; p.err = err;
   p.n_tokens = n_tokens; p.n_reqs = n_reqs; p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads; p.k_dim = k_dim;
   p.v_dim = v_dim; p.page_size = page_size; p.max_pages = max_pages; p.num_pages = num_pages;
-  const int heads_total = n_q_heads + n_kv_heads + (v_off >= 0 ? n_kv_heads : 0);
+  p.norm_after = norm_after; p.maps = maps; p.k_row = k_row; p.v_row = v_row;
+  const int heads_total = n_q_heads + n_kv_heads * maps + (v_off >= 0 ? n_kv_heads : 0);
   const dim3 grid((unsigned)n_tokens, (unsigned)((heads_total + tk::kHeadsWarps - 1) / tk::kHeadsWarps));
   cudaError_t e = cudaSuccess;
-  const bool vec = k_dim % 4 == 0 && v_dim % 4 == 0 && row_stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
+  const bool vec = k_dim % 4 == 0 && v_dim % 4 == 0 && k_row % 4 == 0 && v_row % 4 == 0 && row_stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
                    (v_off < 0 || v_off % 4 == 0);
   if (vec) {
     TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::qkv_heads_vec_kernel<T>, grid, dim3(tk::kHeadsWarps * 32), 0, stream, p));

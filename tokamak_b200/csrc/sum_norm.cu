@@ -9,7 +9,8 @@
 //   1  rows in the activation type
 //   2  the float32 partial sums of a split product
 //   3  the experts' output rows (bfloat16) of a mixture: sum_k weights[t, k] * y[pair_row[t * top + k]]
-//   4  the same with float32 rows, row t * top + k without a list
+//   4  the same with float32 rows
+//      (row t * top + k without a list; a choice of weight 0 is skipped: it may have no row)
 // each formed in float32 in a fixed order before it joins, so a row does not depend on what else is in the step.
 // With a list of rows only those are summed and normed and the stream is left as it is (the model's last norm).
 // One block per row.
@@ -18,7 +19,7 @@
 
 namespace tk {
 
-constexpr int kSumTerms = 2;
+constexpr int kSumTerms = 3;
 
 struct SumTerm {
   const void* data;         // null: no branch
@@ -58,8 +59,9 @@ __device__ __forceinline__ float4 term4(const SumTerm& s, int t, int c, int widt
   }
   for (int k = 0; k < s.count; ++k) {
     const size_t pair = (size_t)t * s.count + k;
-    const size_t row = s.pair_row != nullptr ? (size_t)s.pair_row[pair] : pair;
     const float w = s.weights[pair];
+    if (w == 0.0f) continue;
+    const size_t row = s.pair_row != nullptr ? (size_t)s.pair_row[pair] : pair;
     if (s.kind == 3) acc = axpy4(w, ld4<__nv_bfloat16>((const __nv_bfloat16*)s.data + row * width + c), acc);
     else acc = axpy4(w, ld4<float>((const float*)s.data + row * width + c), acc);
   }
@@ -77,8 +79,9 @@ __device__ __forceinline__ float term1(const SumTerm& s, int t, int c, int width
   }
   for (int k = 0; k < s.count; ++k) {
     const size_t pair = (size_t)t * s.count + k;
-    const size_t row = s.pair_row != nullptr ? (size_t)s.pair_row[pair] : pair;
     const float w = s.weights[pair];
+    if (w == 0.0f) continue;
+    const size_t row = s.pair_row != nullptr ? (size_t)s.pair_row[pair] : pair;
     acc += w * (s.kind == 3 ? __bfloat162float(((const __nv_bfloat16*)s.data)[row * width + c])
                             : ((const float*)s.data)[row * width + c]);
   }
@@ -174,7 +177,8 @@ static bool sum_term_ok(const SumTerm& s) {
 
 TK_API int tk_sum_rmsnorm(float* resid, const void* a, int a_kind, int a_count, long long a_stride, const float* a_weights,
                           const int* a_pair_row, const void* b, int b_kind, int b_count, long long b_stride,
-                          const float* b_weights, const int* b_pair_row, const float* extra, const float* vector,
+                          const float* b_weights, const int* b_pair_row, const void* c, int c_kind, int c_count,
+                          long long c_stride, const float* c_weights, const int* c_pair_row, const float* extra, const float* vector,
                           const float* weight, void* out, const int* rows, int n_rows, int n_tokens, int width, float eps,
                           int dtype, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
@@ -182,15 +186,16 @@ TK_API int tk_sum_rmsnorm(float* resid, const void* a, int a_kind, int a_count, 
   p.resid = resid;
   p.term[0] = tk::SumTerm{a, a_kind, a_count, a_stride, a_weights, a_pair_row};
   p.term[1] = tk::SumTerm{b, b_kind, b_count, b_stride, b_weights, b_pair_row};
+  p.term[2] = tk::SumTerm{c, c_kind, c_count, c_stride, c_weights, c_pair_row};
   p.extra = extra; p.vector = vector; p.weight = weight; p.out = out; p.rows = rows;
   p.n_rows = n_rows; p.n_tokens = n_tokens; p.width = width; p.eps = eps;
   if (resid == nullptr || weight == nullptr || out == nullptr || width < 1 || !tk::sum_term_ok(p.term[0]) ||
-      !tk::sum_term_ok(p.term[1]) || (size_t)width * sizeof(float) > 200 * 1024) {
+      !tk::sum_term_ok(p.term[1]) || !tk::sum_term_ok(p.term[2]) || (size_t)width * sizeof(float) > 200 * 1024) {
     return (int)cudaErrorInvalidValue;
   }
   cudaError_t e = cudaSuccess;
   const int chunks = width / 4;
-  if (width % 4 == 0 && a_stride % 4 == 0 && b_stride % 4 == 0 && chunks <= 512 * tk::kSumPieces) {
+  if (width % 4 == 0 && a_stride % 4 == 0 && b_stride % 4 == 0 && c_stride % 4 == 0 && chunks <= 512 * tk::kSumPieces) {
     // few rows get a thread per piece of four columns, many rows two pieces a thread
     int threads = ((n_rows <= 296 ? chunks : (chunks + 1) / 2) + 31) / 32 * 32;
     if (threads > 512) threads = 512;

@@ -424,7 +424,9 @@ class GatedAttentionSpec:
     position spec whose part rotates neighbouring pairs or halves, or ``none``.  ``q_temp`` ``(coef, every)``: the
     query at position ``p`` is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``softcap``: scores
     are bounded by ``cap * tanh(s / cap)``.  ``unit_sink``: one is added to every softmax denominator (a sink of
-    score 0 without a value).  ``rel_far``: a learned bias ``rel[bucket(i - j), h]`` joins the score, see
+    score 0 without a value); ``sinks``: a learned number per query head, the sink's score.  ``norm_after``: the head
+    norm follows the rotation.  ``pad_rows``: in bfloat16 the rows of the cache get a size that the tiled attention kernels
+    take (``ops.attention_row``), the rest of a row zero; not with a gate.  ``rel_far``: a learned bias ``rel[bucket(i - j), h]`` joins the score, see
     :func:`bucketed_distance_table`; the table's rows are read from the checkpoint.  ``gate``: ``"head"`` (one
     sigmoid gate per head) or ``"channel"`` (one per output channel) or ``None``.  The ``*_name`` fields are the
     tensors' names after the part's prefix."""
@@ -443,6 +445,9 @@ class GatedAttentionSpec:
     q_temp: tuple | None = None
     softcap: float | None = None
     unit_sink: bool = False
+    sinks: bool = False
+    norm_after: bool = False
+    pad_rows: bool = False
     rel_far: int | None = None
     rel_rows: int | None = None
     gate: str | None = None
@@ -453,6 +458,7 @@ class GatedAttentionSpec:
     o_name: str = "o"
     gate_name: str = "g"
     rel_name: str = "rel"
+    sink_name: str = "sink"
     bias_suffix: str = ".b"
     norm_suffix: str = ".norm"
     kind: str = "attention_gated"
@@ -462,7 +468,7 @@ class GatedAttentionSpec:
 class GatedAttention:
     """Grouped-query attention over paged keys and values; query head ``h`` reads key/value head
     ``h // (Hq / Hkv)``; ``score = (q . k) * scale``, capped, plus the distance bias; causal; the softmax
-    denominator may hold one more term ``exp(0)``; the heads are gated by ``sigmoid(W_g h)`` before the output
+    denominator may hold one more term, ``exp(0)`` or the exponential of a learned number per head; the heads are gated by ``sigmoid(W_g h)`` before the output
     projection.
 
     The q, k, v and gate matrices are one stacked operand.  Biases, head norms, the query temperature, the
@@ -481,6 +487,10 @@ class GatedAttention:
             raise ValueError("values that are the keys have the keys' size")
         if spec.gate not in (None, "head", "channel"):
             raise ValueError(f"gate must be None, 'head' or 'channel', got {spec.gate!r}")
+        if spec.unit_sink and spec.sinks:
+            raise ValueError("a sink is either learned or of score 0")
+        if spec.pad_rows and (spec.gate is not None or spec.values_from_keys):
+            raise ValueError("padded rows go with neither a gate nor values that are the keys")
         self.spec = spec
         self.rt = rt
         t = lambda name: tensors[prefix + name]
@@ -501,13 +511,23 @@ class GatedAttention:
         self.q_norm = vec(spec.q_name + spec.norm_suffix) if normed else None
         self.k_norm = vec(spec.k_name + spec.norm_suffix) if normed else None
         self.sinks = torch.zeros(spec.num_heads, dtype=torch.float32, device=rt.device) if spec.unit_sink else None
+        if spec.sinks:
+            self.sinks = vec(spec.sink_name)
         self.dist_bias = bucketed_distance_table(t(spec.rel_name), spec.rel_far) if spec.rel_far is not None else None
         self.position = POSITIONS.get(spec.position.kind)(spec.position, tensors, rt)
         if not hasattr(self.position, "rotary_table"):
             raise ValueError(f"position encoding {spec.position.kind!r} does not rotate queries and keys")
         self.halves = getattr(self.position, "PAIRING", "halves") == "halves"
+        self.k_row, self.v_row = spec.head_dim, spec.v_head_dim
+        if spec.pad_rows and rt.dtype == torch.bfloat16:
+            row = ops.attention_row(max(spec.head_dim, spec.v_head_dim), rt.dtype)
+            if row in ops.ATTENTION_ROWS:
+                self.k_row = self.v_row = row
         self.w_o = t(spec.o_name)
-        self.out_width = spec.num_heads * spec.v_head_dim
+        if self.v_row != spec.v_head_dim:       # the attention rows' padding meets zero columns
+            w = self.w_o.view(-1, spec.num_heads, spec.v_head_dim)
+            self.w_o = torch.nn.functional.pad(w, (0, self.v_row - spec.v_head_dim)).flatten(1).contiguous()
+        self.out_width = spec.num_heads * self.v_row
         self.prefill_heads = spec.num_heads
 
     @staticmethod
@@ -526,6 +546,8 @@ class GatedAttention:
             out[prefix + spec.k_name + spec.norm_suffix] = TensorReq((d,), role="vector")
         if spec.rel_far is not None:
             out[prefix + spec.rel_name] = TensorReq((spec.rel_rows, spec.num_heads), role="bias")
+        if spec.sinks:
+            out[prefix + spec.sink_name] = TensorReq((spec.num_heads,), role="bias")
         if spec.gate is not None:
             out[prefix + spec.gate_name] = TensorReq((spec.num_heads if spec.gate == "head" else spec.num_heads * dv, h))
         out[prefix + spec.o_name] = TensorReq((h, spec.num_heads * dv))
@@ -533,8 +555,8 @@ class GatedAttention:
         return out
 
     def cache_need(self) -> KVPagesNeed:
-        s = self.spec
-        return KVPagesNeed(s.num_kv_heads, s.head_dim, s.window, None if s.v_head_dim == s.head_dim else s.v_head_dim)
+        return KVPagesNeed(self.spec.num_kv_heads, self.k_row, self.spec.window,
+                           None if self.v_row == self.k_row else self.v_row)
 
     def GRAPH_SAFE(self) -> bool:
         return graph_safe(self.position)
@@ -553,15 +575,16 @@ class GatedAttention:
         n = h.shape[0]
         if proj is None:
             proj, proj_off = linear(h, self.w_in, err=step.err), 0
-        q = torch.empty((n, spec.num_heads, spec.head_dim), dtype=h.dtype, device=h.device)
+        q = torch.empty((n, spec.num_heads, self.k_row), dtype=h.dtype, device=h.device)
         table, rotary_dim = self.position.rotary_table(step)
         coef, every = spec.q_temp if spec.q_temp is not None else (0.0, 0)
         ops.qkv_heads(proj, q, cache_view.k, cache_view.v, step, cache_view.table, q_off=proj_off + self.q_off,
                       k_off=proj_off + self.k_off, v_off=None if self.v_off is None else proj_off + self.v_off,
                       q_bias=self.q_bias, k_bias=self.k_bias, v_bias=self.v_bias,
                       head_norm_eps=spec.head_norm_eps, q_norm=self.q_norm, k_norm=self.k_norm, table=table,
-                      rotary_dim=rotary_dim, halves=self.halves, temp_coef=coef, temp_every=every)
-        att = torch.empty((n, spec.num_heads, spec.v_head_dim), dtype=h.dtype, device=h.device)
+                      rotary_dim=rotary_dim, halves=self.halves, temp_coef=coef, temp_every=every, norm_after=spec.norm_after,
+                      k_dim=spec.head_dim, v_dim=spec.v_head_dim)
+        att = torch.empty((n, spec.num_heads, self.v_row), dtype=h.dtype, device=h.device)
         paged_attention(q, att, cache_view, step, scale=spec.softmax_scale, window=spec.window, softcap=spec.softcap,
                         sinks=self.sinks, dist_bias=self.dist_bias)
         att = att.view(n, self.out_width)

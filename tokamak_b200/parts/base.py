@@ -85,8 +85,8 @@ something else joins the stream between two blocks (:class:`~tokamak_b200.models
 :class:`SumBranch` pending.  A norm with ``TAKES_SUM = True`` adds all of it to the stream and normalises in one
 kernel; in front of any other norm the model adds it first (:meth:`SumBranch.settle`).  A feed-forward with
 ``LEAVES_WEIGHTED_ROWS = True`` takes ``combine=False`` and may return
-:class:`~tokamak_b200.csrc.ops.WeightedRows` (a mixture's rows before their weighted sum), which can be a term of a
-``SumBranch``.  An embedding with ``TAKES_KEEP = True`` takes ``keep=``, a float32 tensor for a second copy of its rows.
+:class:`~tokamak_b200.csrc.ops.WeightedRows` (a mixture's rows before their weighted sum) or a tuple of them, which can
+be terms of a ``SumBranch``.  An embedding with ``TAKES_KEEP = True`` takes ``keep=``, a float32 tensor for a second copy of its rows.
 
 ``TAKES_PROJ = True`` (a mixer that can be half of a ``parallel`` mixer): its stacked input projection is ``w_in``
 and its ``branch`` takes ``proj=, proj_off=``, a product of the shared input that holds its columns from
@@ -216,6 +216,17 @@ class NormedBranch:
     eps: float
     layer_scale: torch.Tensor | None = None
     groups: int = 1
+
+
+@dataclass
+class NormedSum:
+    """Two branches that join the residual stream together, each after a norm of its own:
+    ``resid += rmsnorm(x_1, eps) * weight_1 + rmsnorm(x_2, eps) * weight_2`` (a factor on a branch is part of its weight).
+    ``x_1`` and ``x_2`` are what :func:`linear` returned.  The norm that consumes it
+    (:meth:`RMSNorm.add_norm <tokamak_b200.parts.norm.RMSNorm.add_norm>`) does all of it in one kernel."""
+
+    first: NormedBranch
+    second: NormedBranch
 
 
 @dataclass

@@ -15,7 +15,8 @@ class PreNormBlockSpec:
     """One block and the checkpoint names of its tensors.
 
     ``mixer_prefix`` and ``ffn_prefix`` end with a dot; ``norm1_name`` and
-    ``norm2_name`` are full tensor names.
+    ``norm2_name`` are full tensor names.  ``feed_forward`` of ``None`` is a block of one sublayer (``norm2`` and the
+    two names are then not looked at).
     """
 
     name: str
@@ -25,8 +26,8 @@ class PreNormBlockSpec:
     feed_forward: object
     norm1_name: str
     mixer_prefix: str
-    norm2_name: str
-    ffn_prefix: str
+    norm2_name: str | None
+    ffn_prefix: str | None
     kind: str = "pre_norm"
 
 
@@ -42,8 +43,9 @@ class PreNormBlock:
 
     Where a branch can, its last product adds itself to the residual stream and prepares
     the input of the norm after it (see ``parts/base.py``, owed norms): the mixer for
-    ``norm2``, the feed-forward for ``next_norm``, the norm that will consume what this
-    block leaves pending.
+    ``norm2``, the feed-forward (or, in a block without one, the mixer) for ``next_norm``, the norm
+    that will consume what this block leaves pending.  A feed-forward that can leave several terms (the rows of a
+    mixture of experts in front of their weighted sum) leaves them to that norm as a :class:`SumBranch`.
     """
 
     TAKES_NEXT_NORM = True
@@ -52,25 +54,31 @@ class PreNormBlock:
         self.spec = spec
         self.norm1 = NORMS.get(spec.norm1.kind)(spec.norm1, spec.norm1_name, tensors, rt)
         self.mixer = MIXERS.get(spec.mixer.kind)(spec.mixer, spec.mixer_prefix, tensors, rt)
-        self.norm2 = NORMS.get(spec.norm2.kind)(spec.norm2, spec.norm2_name, tensors, rt)
-        self.feed_forward = FEED_FORWARDS.get(spec.feed_forward.kind)(
-            spec.feed_forward, spec.ffn_prefix, tensors, rt)
+        self.norm2 = self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.norm2 = NORMS.get(spec.norm2.kind)(spec.norm2, spec.norm2_name, tensors, rt)
+            self.feed_forward = FEED_FORWARDS.get(spec.feed_forward.kind)(
+                spec.feed_forward, spec.ffn_prefix, tensors, rt)
 
     @staticmethod
     def expected_tensors(spec: PreNormBlockSpec) -> dict[str, TensorReq]:
         out: dict[str, TensorReq] = {}
         out.update(NORMS.get(spec.norm1.kind).expected_tensors(spec.norm1, spec.norm1_name))
         out.update(MIXERS.get(spec.mixer.kind).expected_tensors(spec.mixer, spec.mixer_prefix))
-        out.update(NORMS.get(spec.norm2.kind).expected_tensors(spec.norm2, spec.norm2_name))
-        out.update(FEED_FORWARDS.get(spec.feed_forward.kind).expected_tensors(
-            spec.feed_forward, spec.ffn_prefix))
+        if spec.feed_forward is not None:
+            out.update(NORMS.get(spec.norm2.kind).expected_tensors(spec.norm2, spec.norm2_name))
+            out.update(FEED_FORWARDS.get(spec.feed_forward.kind).expected_tensors(
+                spec.feed_forward, spec.ffn_prefix))
         return out
 
     def cache_need(self):
         return self.mixer.cache_need()
 
+    def _parts(self) -> list:
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None]
+
     def GRAPH_SAFE(self) -> bool:
-        return graph_safe(self.norm1, self.mixer, self.norm2, self.feed_forward)
+        return graph_safe(*self._parts())
 
     @property
     def prefill_heads(self) -> int | None:
@@ -78,7 +86,7 @@ class PreNormBlock:
         return getattr(self.mixer, "prefill_heads", None)
 
     def weight_bytes(self) -> int:
-        return weight_bytes(self.norm1, self.mixer, self.norm2, self.feed_forward)
+        return weight_bytes(*self._parts())
 
     @property
     def entry_norm(self):
@@ -94,10 +102,22 @@ class PreNormBlock:
 
     def forward(self, resid: torch.Tensor, pending, step, cache_view, next_norm=None):
         h = self.norm1.add_norm(resid, pending)
+        then = (resid, next_norm) if next_norm is not None else None
+        if self.feed_forward is None:
+            return resid, self._branch(self.mixer, h, (step, cache_view), then)
         a = self._branch(self.mixer, h, (step, cache_view), (resid, self.norm2))
         h = self.norm2.add_norm(resid, a)
-        out = self._branch(self.feed_forward, h, (step,), (resid, next_norm) if next_norm is not None else None)
-        return resid, out
+        if getattr(self.feed_forward, "LEAVES_WEIGHTED_ROWS", False):
+            return resid, SumBranch(self._terms(self.feed_forward, h, step))
+        return resid, self._branch(self.feed_forward, h, (step,), then)
+
+    @staticmethod
+    def _terms(feed_forward, h, step) -> tuple:
+        """What a feed-forward that may leave several terms leaves, as a tuple."""
+        if isinstance(h, OwedNorm) and not getattr(feed_forward, "TAKES_OWED_NORM", False):
+            h = h.materialize()
+        out = feed_forward.forward(h, step, combine=False)
+        return out if isinstance(out, tuple) else (out,)
 
 
 @dataclass(frozen=True)
@@ -436,6 +456,8 @@ class ParallelBlock:
             h = h.materialize()
         terms = [self.mixer.forward(h, step, cache_view)]
         if self.feed_forward is not None:
-            kw = {"combine": False} if getattr(self.feed_forward, "LEAVES_WEIGHTED_ROWS", False) else {}
-            terms.append(self.feed_forward.forward(h, step, **kw))
+            if getattr(self.feed_forward, "LEAVES_WEIGHTED_ROWS", False):
+                terms += PreNormBlock._terms(self.feed_forward, h, step)
+            else:
+                terms.append(self.feed_forward.forward(h, step))
         return resid, SumBranch(tuple(terms))

@@ -102,8 +102,8 @@ class SwiGLU:
 
 @dataclass(frozen=True)
 class MlpSpec:
-    """An ungated unit ``down(act(up(x)))``; ``activation`` is ``relu2`` (the square of relu), ``gelu_tanh`` or
-    ``silu``; the names are the tensors' names after the part's prefix."""
+    """An ungated unit ``down(act(up(x)))``; ``activation`` is ``relu2`` (the square of relu), ``gelu`` (exact),
+    ``gelu_tanh`` or ``silu``; the names are the tensors' names after the part's prefix."""
 
     hidden_size: int
     intermediate_size: int
@@ -161,9 +161,17 @@ class MoESpec:
     """A mixture of ``num_experts`` units of inner size ``intermediate_size`` of which every token uses ``top``.
     ``gated``: a unit is ``down(act(gate(x)) * up(x))`` with ``activation`` ``silu`` or ``gelu_tanh``; otherwise
     ``down(act(up(x)))`` with ``relu2``, ``silu`` or ``gelu_tanh``.  ``router``: ``sigmoid`` (the weights are the chosen
-    experts' plain scores) or ``softmax`` (the softmax over the chosen experts' logits only).  The experts form ``num_groups`` equal groups of neighbours and only experts of the ``keep_groups``
-    best groups can be chosen (``num_groups = keep_groups = 1``: no restriction).  ``correction``: a learned
-    number per expert that is added to the scores for the choice only.  The ``*_name`` fields are the
+    experts' plain scores), ``softmax`` (the softmax over the chosen experts' logits only) or ``softmax_all`` (the softmax
+    over all outputs).  ``normalize``: the chosen scores are divided by their sum (+ 1e-20).  The experts form
+    ``num_groups`` equal groups of neighbours and only experts of the ``keep_groups`` best groups can be chosen
+    (``num_groups = keep_groups = 1``: no restriction); ``group_score``: a group's score is the sum of its two largest
+    choice scores (``top2``) or its largest (``best``).  ``correction``: a learned number per expert that is added to the
+    scores for the choice only.
+
+    ``identity``: the router has so many outputs more, whose experts hand the input on (no tensors; they are in the
+    scores, groups and choice like the others).  ``shared_size``: one more unit of that inner size under
+    ``shared_prefix`` runs for every token, times ``sigmoid(W_sg h)``, one number per token.  ``pad_inner``: in bfloat16 an
+    inner size that the grouped tensor-core products do not take is filled up with zeros.  The ``*_name`` fields are the
     tensors' names after the part's prefix; expert ``e``'s matrices lie under ``expert_prefix.format(e)``."""
 
     hidden_size: int
@@ -175,6 +183,11 @@ class MoESpec:
     correction: bool = True
     gated: bool = True
     router: str = "sigmoid"
+    normalize: bool = False
+    group_score: str = "top2"
+    identity: int = 0
+    shared_size: int | None = None
+    pad_inner: bool = False
     activation: str = "silu"
     router_name: str = "router"
     correction_name: str = "correction"
@@ -182,6 +195,8 @@ class MoESpec:
     gate_name: str = "gate"
     up_name: str = "up"
     down_name: str = "down"
+    shared_prefix: str = "shared."
+    shared_gate_name: str = "sg"
     kind: str = "moe"
 
 
@@ -199,6 +214,11 @@ class MixtureOfExperts:
     out expert by expert on the device, so nothing is read back and a step of single tokens can be
     replayed from a CUDA graph; the products run over tiles of one expert's rows (``csrc/moe.cu``).  The
     result is float32 and does not depend on what else is in the batch.
+
+    A shared expert is cut along its inner size into pieces of an expert's (the last one filled up with zeros); a
+    unit's output is the sum of its pieces', so the pieces are experts behind the others that every token chooses,
+    and the shared expert costs no launches of its own.  Its gate is one more row of the router.  The identity
+    experts' share of the output is one more term, the input times a number per token.
     """
 
     GRAPH_SAFE = True
@@ -210,25 +230,41 @@ class MixtureOfExperts:
             raise ValueError(f"unknown activation {spec.activation!r}; known: {', '.join(known)}")
         if spec.router not in ops.ROUTER_KINDS:
             raise ValueError(f"unknown router {spec.router!r}; known: {', '.join(ops.ROUTER_KINDS)}")
-        if spec.num_experts % spec.num_groups or not 1 <= spec.keep_groups <= spec.num_groups:
-            raise ValueError(f"{spec.num_experts} experts do not form {spec.num_groups} equal groups of which "
+        outputs = spec.num_experts + spec.identity
+        if outputs % spec.num_groups or not 1 <= spec.keep_groups <= spec.num_groups:
+            raise ValueError(f"{outputs} experts do not form {spec.num_groups} equal groups of which "
                              f"{spec.keep_groups} are kept")
-        if not 1 <= spec.top <= spec.keep_groups * (spec.num_experts // spec.num_groups):
+        if not 1 <= spec.top <= spec.keep_groups * (outputs // spec.num_groups):
             raise ValueError(f"{spec.top} experts cannot be chosen from {spec.keep_groups} groups of "
-                             f"{spec.num_experts // spec.num_groups}")
+                             f"{outputs // spec.num_groups}")
         self.spec = spec
         self.rt = rt
-        self.router = tensors[prefix + spec.router_name].float().contiguous()
+        self.router = tensors[prefix + spec.router_name].float()
         self.correction = tensors[prefix + spec.correction_name].contiguous() if spec.correction else None
-        stack = lambda name: torch.stack([tensors[prefix + spec.expert_prefix.format(e) + name]
-                                          for e in range(spec.num_experts)]).contiguous()
-        self.w_gate = stack(spec.gate_name) if spec.gated else None
-        self.w_up, self.w_down = stack(spec.up_name), stack(spec.down_name)
+        ff = spec.intermediate_size
+        if spec.pad_inner and rt.dtype == torch.bfloat16 and ops.PAIR_GEMM_POLICY != "off":
+            ff += -ff % (ops.SWIGLU_TILE_BLOCK if spec.gated else 8)
+        self.inner = ff
+        self.shared = 0 if spec.shared_size is None else -(-spec.shared_size // ff)      # pieces of the shared expert
+        names = ([spec.gate_name] if spec.gated else []) + [spec.up_name, spec.down_name]
+        stacked = {}
+        for name in names:
+            dim = 1 if name == spec.down_name else 0       # the inner size's place in the matrix
+            fill = lambda m, size: torch.nn.functional.pad(m, (0, size - m.shape[1]) if dim else (0, 0, 0, size - m.shape[0]))
+            mats = [fill(tensors[prefix + spec.expert_prefix.format(e) + name], ff) for e in range(spec.num_experts)]
+            if self.shared:
+                mats += fill(tensors[prefix + spec.shared_prefix + name], self.shared * ff).split(ff, dim=dim)
+            stacked[name] = torch.stack(mats).contiguous()
+        if self.shared:
+            self.router = torch.cat([self.router, tensors[prefix + spec.shared_prefix + spec.shared_gate_name].float()])
+        self.router = self.router.contiguous()
+        self.w_gate = stacked[spec.gate_name] if spec.gated else None
+        self.w_up, self.w_down = stacked[spec.up_name], stacked[spec.down_name]
         # bfloat16 at sizes the product on pairs of SMs takes: gate and up rows alternate in blocks, so that
         # the activation is the product's epilogue (an ungated unit's first matrix is taken as it is); the
         # matrices are then kept only in that form
         self.w_first = None
-        if ops.moe_tc_takes(self.w_up.dtype, spec.hidden_size, spec.intermediate_size, spec.gated):
+        if ops.moe_tc_takes(self.w_up.dtype, spec.hidden_size, ff, spec.gated):
             self.w_first = ops.moe_stack_gate_up(self.w_gate, self.w_up) if spec.gated else self.w_up
             self.w_gate = self.w_up = None
 
@@ -242,29 +278,44 @@ class MixtureOfExperts:
                 out[p + spec.gate_name] = TensorReq((i, h))
             out[p + spec.up_name] = TensorReq((i, h))
             out[p + spec.down_name] = TensorReq((h, i))
-        out[prefix + spec.router_name] = TensorReq((spec.num_experts, h), role="matrix_f32")
+        outputs = spec.num_experts + spec.identity
+        out[prefix + spec.router_name] = TensorReq((outputs, h), role="matrix_f32")
         if spec.correction:
-            out[prefix + spec.correction_name] = TensorReq((spec.num_experts,), role="bias")
+            out[prefix + spec.correction_name] = TensorReq((outputs,), role="bias")
+        if spec.shared_size is not None:
+            p = prefix + spec.shared_prefix
+            for name in ([spec.gate_name] if spec.gated else []) + [spec.up_name]:
+                out[p + name] = TensorReq((spec.shared_size, h))
+            out[p + spec.down_name] = TensorReq((h, spec.shared_size))
+            out[p + spec.shared_gate_name] = TensorReq((1, h), role="matrix_f32")
         return out
 
     def weight_bytes(self) -> int:
-        """What a step of one token reads: the router and ``top`` experts (a large step reads all)."""
-        per_expert = tensor_bytes(self.w_gate, self.w_up, self.w_first, self.w_down) // self.spec.num_experts
-        return tensor_bytes(self.router, self.correction) + self.spec.top * per_expert
+        """What a step of one token reads: the router, ``top`` experts and the shared one (a large step reads all)."""
+        per_expert = tensor_bytes(self.w_gate, self.w_up, self.w_first, self.w_down) // self.w_down.shape[0]
+        return tensor_bytes(self.router, self.correction) + (self.spec.top + self.shared) * per_expert
 
     def forward(self, h, step, combine: bool = True):
+        """float32 sums ``[1, tokens, width]``; with ``combine=False`` the :class:`~tokamak_b200.csrc.ops.WeightedRows` in
+        front of the sum, or a tuple of them."""
         spec = self.spec
         if isinstance(h, OwedNorm):
             h = h.materialize()
         tc = self.w_first is not None
         routing = ops.moe_route(h, self.router, self.correction, top=spec.top, n_groups=spec.num_groups,
-                                keep=spec.keep_groups, padded=tc, kind=spec.router)
+                                keep=spec.keep_groups, padded=tc, kind=spec.router, group_score=spec.group_score,
+                                normalize=spec.normalize, identity=spec.identity, shared=self.shared)
         kw = dict(activation=spec.activation, combine=combine)
-        if tc and ops.moe_small_takes(h.shape[0], spec.top, spec.hidden_size, spec.intermediate_size, spec.gated):
+        if tc and ops.moe_small_takes(h.shape[0], spec.top + self.shared, spec.hidden_size, self.inner, spec.gated):
             out = ops.moe_experts_small(h, routing, self.w_first, self.w_down, gated=spec.gated, **kw)
         elif tc:
             out = ops.moe_experts_tc(h, routing, self.w_first, self.w_down, step.err, gated=spec.gated, **kw)
         else:
             out = ops.moe_experts(h, routing, self.w_gate, self.w_up, self.w_down, **kw)
+        own = ops.WeightedRows(h, routing.identity_weight, None) if spec.identity else None
+        if not combine:
+            return out if own is None else (out, own)
+        if own is not None:
+            out = out + own.combine()
         # float32 sums, one part: the consuming norm reads them as they are
-        return out.unsqueeze(0) if combine else out
+        return out.unsqueeze(0)

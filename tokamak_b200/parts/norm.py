@@ -7,7 +7,7 @@ from dataclasses import dataclass
 import torch
 
 from ..csrc import ops
-from .base import NORMS, HyperBranch, NormedBranch, OwedNorm, Runtime, SumBranch, TensorReq
+from .base import NORMS, HyperBranch, NormedBranch, NormedSum, OwedNorm, Runtime, SumBranch, TensorReq
 
 
 @dataclass(frozen=True)
@@ -53,7 +53,7 @@ class RMSNorm:
         normalised and ``resid`` is left as it is.  ``delta`` may be an
         :class:`OwedNorm`: the branch has been added to ``resid`` already; if it was
         prepared for this norm it is handed on as it is (its consumer pays the scale).
-        A :class:`NormedBranch` is normalised, scaled and added by the same kernel; all of a
+        A :class:`NormedBranch` (or the two of a :class:`NormedSum`) is normalised, scaled and added by the same kernel; all of a
         :class:`SumBranch` joins in one.
         """
         if isinstance(delta, NormedBranch):
@@ -61,6 +61,12 @@ class RMSNorm:
             out = torch.empty((n, self.spec.dim), dtype=self.rt.dtype, device=resid.device)
             ops.branch_norm_add(resid, delta.x, delta.weight, delta.layer_scale, delta.eps, self.weight, out,
                                 self.spec.eps, rows, branch_groups=delta.groups)
+            return out
+        if isinstance(delta, NormedSum):
+            n = rows.numel() if rows is not None else resid.shape[0]
+            out = torch.empty((n, self.spec.dim), dtype=self.rt.dtype, device=resid.device)
+            a, b = delta.first, delta.second
+            ops.branch_pair_norm_add(resid, a.x, a.weight, b.x, b.weight, a.eps, self.weight, out, self.spec.eps, rows)
             return out
         if isinstance(delta, SumBranch):
             n = rows.numel() if rows is not None else resid.shape[0]

@@ -73,6 +73,18 @@ class YarnScaling:
 
 
 @dataclass(frozen=True)
+class WaveScaling:
+    """Stretching of a rotary encoding by wavelength, as in Llama 3.1: a pair that turns more than ``high`` times over
+    ``original`` positions keeps its frequency, one that turns fewer than ``low`` times has it divided by ``factor``,
+    those between get a linear blend of the two; cosine and sine keep their size."""
+
+    factor: float
+    original: float
+    low: float
+    high: float
+
+
+@dataclass(frozen=True)
 class RopePairsSpec:
     """Rotation of neighbouring pairs (elements 2i and 2i+1) over the first ``rotary_dim``
     elements of a head; the rest passes unrotated.  ``yarn`` stretches the frequencies."""
@@ -100,6 +112,25 @@ def yarn_frequencies(rotary_dim: int, theta: float, yarn: YarnScaling | None) ->
     hi = min(math.ceil(where(yarn.slow)), rotary_dim - 1)
     ramp = ((idx / 2 - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
     return freq / yarn.factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(yarn.factor) + 1.0
+
+
+def wave_frequencies(rotary_dim: int, theta: float, wave: WaveScaling) -> tuple[torch.Tensor, float]:
+    """``(float64 frequencies [rotary_dim / 2], 1.0)``.  A pair of frequency ``f0`` turns ``t = original f0 / (2 pi)``
+    times over the original length; with ``s = (t - low) / (high - low)``: ``f0`` where ``t > high``, ``f0 / factor``
+    where ``t < low``, else ``(1 - s) f0 / factor + s f0``."""
+    import math
+    freq, _ = yarn_frequencies(rotary_dim, theta, None)
+    turns = wave.original * freq / (2.0 * math.pi)
+    span = wave.high - wave.low
+    s = ((turns - wave.low) / span).clamp(0.0, 1.0) if span > 0 else (turns >= wave.low).to(torch.float64)
+    return (1.0 - s) * freq / wave.factor + s * freq, 1.0
+
+
+def scaled_frequencies(rotary_dim: int, theta: float, scaling) -> tuple[torch.Tensor, float]:
+    """Frequencies and the factor on cosine and sine for a :class:`YarnScaling`, a :class:`WaveScaling` or ``None``."""
+    if isinstance(scaling, WaveScaling):
+        return wave_frequencies(rotary_dim, theta, scaling)
+    return yarn_frequencies(rotary_dim, theta, scaling)
 
 
 @POSITIONS.register("rope_pairs")
@@ -136,18 +167,21 @@ class RopePairs:
 @dataclass(frozen=True)
 class RopeHalvesSpec:
     """Rotation of halves (elements i and i + rotary_dim / 2) over the first ``rotary_dim`` elements of a head;
-    the rest passes unrotated.  ``linear_factor`` divides every frequency."""
+    the rest passes unrotated.  ``linear_factor`` divides every frequency; ``scaling`` (:class:`YarnScaling`,
+    :class:`WaveScaling` or ``None``) stretches them."""
 
     rotary_dim: int
     theta: float
     linear_factor: float = 1.0
+    scaling: object = None
     kind: str = "rope_halves"
 
 
 @POSITIONS.register("rope_halves")
 class RopeHalves:
     """Rotary embedding in the half-split layout on part of the head: element ``i < rotary_dim / 2`` and element
-    ``i + rotary_dim / 2`` turn by ``position * theta ** (-2i / rotary_dim) / linear_factor``.  The frequencies are
+    ``i + rotary_dim / 2`` turn by ``position * theta ** (-2i / rotary_dim) / linear_factor`` (or by a stretched
+    frequency, see the spec's ``scaling``; YaRN also scales cosine and sine).  The frequencies are
     formed in float64 and rounded to float32 once; position times frequency, cosine and sine are float32, once
     per step.  The mixer's kernel does the rotation (``PAIRING`` tells it which elements pair up)."""
 
@@ -158,7 +192,7 @@ class RopeHalves:
         if spec.rotary_dim % 2 or spec.rotary_dim < 0:
             raise ValueError(f"the rotated part of a head must be even, got {spec.rotary_dim}")
         self.spec = spec
-        freq, _ = yarn_frequencies(spec.rotary_dim, spec.theta, None)
+        freq, self.magnitude = scaled_frequencies(spec.rotary_dim, spec.theta, spec.scaling)
         self.inv_freq = (freq / spec.linear_factor).to(torch.float32).to(rt.device)
 
     @staticmethod
@@ -171,7 +205,7 @@ class RopeHalves:
         key = ("rope_table", self.spec)
         table = step.scratch.get(key)
         if table is None:
-            table = ops.rope_table(step.positions, self.inv_freq)
+            table = ops.rope_table(step.positions, self.inv_freq, self.magnitude)
             step.scratch[key] = table
         return table, self.spec.rotary_dim
 
