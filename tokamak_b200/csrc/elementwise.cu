@@ -422,7 +422,7 @@ TK_API int tk_swiglu(const void* gate_up, const float* parts, int n_parts, long 
 TK_API int tk_unary_act(const void* x, const float* parts, int n_parts, long long part_stride, void* out,
                         long long total, int dtype, int act, cudaStream_t stream) {
   if (total <= 0) return 0;
-  if ((x == nullptr) == (parts == nullptr) || act < 0 || act > 2) return (int)cudaErrorInvalidValue;
+  if ((x == nullptr) == (parts == nullptr) || act < 0 || act > 3) return (int)cudaErrorInvalidValue;
   size_t blocks = ((size_t)total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   cudaError_t e = cudaSuccess;
