@@ -136,17 +136,20 @@ class GatedDeltaRule:
             prefix + spec.beta_name: TensorReq((hh, w)),
             prefix + spec.decay_log_name: TensorReq((hh,), role="bias"),
             prefix + spec.norm_name: TensorReq((spec.value_dim,), role="vector"),
-            prefix + spec.o_name: TensorReq((w, hv)),
         }
         per_head = hh if spec.decay_rank is None else hh * spec.key_dim
+        if spec.decay_rank is None:
+            out[prefix + spec.decay_name] = TensorReq((per_head, w))
+        else:
+            out[prefix + spec.decay_names[0]] = TensorReq((spec.decay_rank, w))
+            out[prefix + spec.decay_names[1]] = TensorReq((per_head, spec.decay_rank))
         out[prefix + spec.decay_bias_name] = TensorReq((per_head,), role="bias")
-        for rank, name, names, rows in ((spec.decay_rank, spec.decay_name, spec.decay_names, per_head),
-                                        (spec.gate_rank, spec.gate_name, spec.gate_names, hv)):
-            if rank is None:
-                out[prefix + name] = TensorReq((rows, w))
-            else:
-                out[prefix + names[0]] = TensorReq((rank, w))
-                out[prefix + names[1]] = TensorReq((rows, rank))
+        if spec.gate_rank is None:
+            out[prefix + spec.gate_name] = TensorReq((hv, w))
+        else:
+            out[prefix + spec.gate_names[0]] = TensorReq((spec.gate_rank, w))
+            out[prefix + spec.gate_names[1]] = TensorReq((hv, spec.gate_rank))
+        out[prefix + spec.o_name] = TensorReq((w, hv))
         return out
 
     def cache_need(self) -> StateNeed:
