@@ -1,0 +1,458 @@
+"""The Sofinex design on the GPU: every mechanism's kernels against the plain implementation, then whole
+models under every way of cutting and batching their requests, and generation through the engine's entry
+point."""
+
+from __future__ import annotations
+
+import functools
+import json
+import math
+import subprocess
+import sys
+import tempfile
+from pathlib import Path
+from types import SimpleNamespace
+
+import numpy as np
+import pytest
+import torch
+
+import sofinex_configs as sc
+import traces
+from helpers import assert_logits_close, random_tokens
+from plain import sofinex_plain as plain
+
+pytestmark = pytest.mark.gpu
+
+ROOT = Path(__file__).resolve().parent.parent
+DTYPES = ["float32", "bfloat16"]
+TORCH = {"float32": torch.float32, "bfloat16": torch.bfloat16}
+_TMP = []
+
+
+@functools.lru_cache(maxsize=None)
+def folder_of(tag: str, dtype: str) -> Path:
+    tmp = tempfile.TemporaryDirectory(prefix=f"sx_{tag}_{dtype}_")
+    _TMP.append(tmp)
+    return Path(sc.write_folder(tmp.name, tag, dtype))
+
+
+@functools.lru_cache(maxsize=None)
+def _truth(folder: str, tokens: tuple):
+    """Logits of the whole sequence, and for every position how close any router came to another choice at
+    or before it (a choice made otherwise early in a sequence reaches later positions through keys and states)."""
+    cfg, w = plain.load_folder(folder)
+    margins = []
+    logits = plain.forward(cfg, w, list(tokens), margins_out=margins)
+    risk = torch.stack(margins).min(0).values.cummin(0).values if margins else torch.full((len(tokens),), math.inf)
+    return logits, risk
+
+
+# bfloat16: a row is judged against what rounding alone costs in its request (the plain implementation
+# rounding at every product's input and output): the level is the worst row of the request, the limit four
+# times that and never below the level of a well-conditioned row.  A wrong key, state or expert moves a row by about
+# its spread.  So does a router that rounding tips elsewhere than in the plain implementation: the few rows
+# beyond the limit that have a router within CLOSE of another choice, at or before them, are let through, counted.
+BF16_FLOOR_RMS, BF16_FLOOR_MAX, BF16_TIMES = 0.05, 0.2, 4.0
+CLOSE, TIPPED_ROWS, TIPPED_SHARE = 0.01, 2, 0.06
+
+
+@functools.lru_cache(maxsize=None)
+def _rounding_level(folder: str, tokens: tuple) -> tuple[float, float]:
+    cfg, w = plain.load_folder(folder)
+    want = _truth(folder, tokens)[0]
+    rounded = plain.forward(cfg, w, list(tokens), ROUND=plain.bf16_round)
+    rel = (rounded - want).abs() / want.std(dim=-1, keepdim=True).clamp_min(1e-6)
+    return rel.pow(2).mean(-1).sqrt().max().item(), rel.max().item()
+
+
+def check_rows(results, rows, reqs, folder, dtype, what) -> int:
+    n, tipped = 0, []
+    for step in sorted(rows):
+        got = torch.from_numpy(np.asarray(results[step])).double()
+        for i, (rid, p) in enumerate(rows[step]):
+            where = f"{what}: step {step}, request {rid!r}, position {p}"
+            toks = tuple(int(t) for t in reqs[rid])
+            logits, risk = _truth(str(folder), toks)
+            want = logits[p]
+            n += 1
+            if dtype == "float32":
+                assert_logits_close(got[i:i + 1], want[None], dtype, where)
+                continue
+            assert torch.isfinite(got[i]).all(), where
+            mine = (got[i] - want).abs() / want.std().clamp_min(1e-6)
+            base_rms, base_max = _rounding_level(str(folder), toks)
+            rms = mine.pow(2).mean().sqrt().item()
+            ok = (rms <= max(BF16_FLOOR_RMS, BF16_TIMES * base_rms)
+                  and mine.max().item() <= max(BF16_FLOOR_MAX, BF16_TIMES * base_max))
+            if not ok and risk[p].item() < CLOSE:
+                tipped.append((rid, p))
+                continue
+            assert ok, (f"{where}: off by {rms:.3e} (rms) and {mine.max().item():.3e} (max) of the row's spread; "
+                        f"rounding alone costs up to {base_rms:.3e} and {base_max:.3e}")
+    assert len(tipped) <= max(TIPPED_ROWS, TIPPED_SHARE * n), f"{what}: {len(tipped)} of {n} rows are off: {tipped}"
+    return n
+
+
+def dev(x, dtype=None):
+    return x.to("cuda", dtype) if dtype is not None else x.to("cuda")
+
+
+def i32(v):
+    return torch.tensor(list(v), dtype=torch.int32, device="cuda")
+
+
+def close(got, want, dtype, scale=1.0):
+    got, want = got.detach().cpu().double(), want.double()
+    tol = (2e-5 if dtype == "float32" else 2e-2) * scale
+    err = (got - want).abs().max().item()
+    assert err <= tol * max(1.0, want.abs().max().item()), f"off by {err:.3e}"
+
+
+def fake_step(q_lens, slots, starts, heads=1):
+    """What a kernel reads of a step: requests of ``q_lens`` tokens in ``slots``, continuing at ``starts``."""
+    from tokamak_b200.csrc import ops
+    tok_req, pos, q_start = [], [], []
+    at = 0
+    for r, (n, s) in enumerate(zip(q_lens, starts)):
+        q_start.append(at)
+        tok_req += [r] * n
+        pos += list(range(s, s + n))
+        at += n
+    kv_len = [s + n for s, n in zip(starts, q_lens)]
+    rec, n_parts, n_split = ops.prefill_tc_records(q_start, q_lens, kv_len, slots, heads=heads,
+                                                   sms=ops.sm_count(torch.device("cuda", 0)))
+    return SimpleNamespace(tok_req=i32(tok_req), positions=i32(pos), req_q_start=i32(q_start), req_q_len=i32(q_lens),
+                           req_slot=i32(slots), req_kv_len=i32(kv_len), max_kv_len=max(kv_len),
+                           err=torch.zeros(4, dtype=torch.int32, device="cuda"), max_q_len=max(q_lens), n_tokens=at,
+                           scratch={}, decode_items=i32([s for s, n in zip(q_start, q_lens) if n == 1]),
+                           prefill_items=i32([s + j for s, n in zip(q_start, q_lens) if n > 1 for j in range(n)]),
+                           prefill_tc=ops.PrefillItems(torch.from_numpy(rec).cuda(), n_parts, n_split),
+                           prefill_tiles=i32([x for r, n in enumerate(q_lens) if n > 1 for t in range(-(-n // 64)) for x in (r, t)]))
+
+
+def run_in_steps(seqs, slots, cuts, fn, heads=1):
+    """Feed sequences (``[T, ...]`` each, one per request) through ``fn(rows of the step, step)`` cut into steps:
+    ``cuts[r]`` lists request r's portion sizes, step by step (0: the request sits the step out).  Returns
+    the outputs put together again per request."""
+    outs = [[] for _ in seqs]
+    fed = [0] * len(seqs)
+    for s in range(max(len(c) for c in cuts)):
+        live = [r for r in range(len(seqs)) if s < len(cuts[r]) and cuts[r][s] > 0]
+        step = fake_step([cuts[r][s] for r in live], [slots[r] for r in live], [fed[r] for r in live], heads)
+        rows = torch.cat([seqs[r][fed[r]:fed[r] + cuts[r][s]] for r in live])
+        y = fn(rows, step)
+        assert step.err.tolist()[0] == 0
+        at = 0
+        for r in live:
+            outs[r].append(y[at:at + cuts[r][s]].detach().cpu())
+            at += cuts[r][s]
+            fed[r] += cuts[r][s]
+    assert fed == [len(x) for x in seqs]
+    return [torch.cat(o) for o in outs]
+
+
+def _part(registry, spec, weights, dtype, prefix="m."):
+    from tokamak_b200.parts.base import Runtime
+    cls = registry.get(spec.kind)
+    tensors = {}
+    for name, req in cls.expected_tensors(spec, prefix).items():
+        t = weights[name[len(prefix):]]
+        assert tuple(t.shape) == tuple(req.shape), name
+        tensors[name] = dev(t, TORCH[dtype] if req.role == "matrix" else torch.float32)
+    return cls(spec, prefix, tensors, Runtime(device=torch.device("cuda"), dtype=TORCH[dtype]))
+
+
+def _rounded(gen, dtype):
+    return lambda *s, std=1.0: (torch.randn(*s, generator=gen) * std).to(TORCH[dtype]).float()
+
+
+def _doubles(w):
+    return {k: t.double() for k, t in w.items()}
+
+
+# ======================================================================= mechanisms alone
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,width,ff", [(3, 48, 72), (1, 128, 256), (40, 128, 384), (70, 54, 50), (600, 256, 11008 // 8), (4500, 64, 1536)])
+def test_dense_feed_forward_with_the_exact_gelu(dtype, n, width, ff):
+    from tokamak_b200.parts.base import FEED_FORWARDS
+    from tokamak_b200.parts.feedforward import MlpSpec
+    gen = torch.Generator().manual_seed(n + ff)
+    rnd = _rounded(gen, dtype)
+    w = {"up": rnd(ff, width, std=1.5 / width ** 0.5), "down": rnd(width, ff, std=1.5 / ff ** 0.5)}
+    x = rnd(n, width)
+    part = _part(FEED_FORWARDS, MlpSpec(width, ff, activation="gelu"), w, dtype)
+    got = part.forward(dev(x, TORCH[dtype]), fake_step([n], [0], [0]))
+    got = got.float().sum(0) if got.dim() == 3 else got.float()
+    close(got, plain.dense_ff(x.double(), _doubles(w)), dtype)
+    from tokamak_b200.csrc import ops
+    z = torch.linspace(-6, 6, 1000).repeat(2, 1)
+    act = ops.unary_act(dev(z), torch.float32, "gelu").cpu().double()
+    assert (act - plain.gelu_exact(z.double())).abs().max() < 1e-6          # the tanh form is off by 4e-4
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,heads,dv,row", [(5, 3, 14, 14), (1, 2, 96, 128), (33, 4, 128, 128), (7, 1, 5, 64), (2, 5, 300, 300)])
+def test_difference_of_two_maps(dtype, n, heads, dv, row):
+    from tokamak_b200.csrc import ops
+    gen = torch.Generator().manual_seed(dv)
+    a = _rounded(gen, dtype)(n, 2 * heads, row)
+    got = ops.map_difference(dev(a, TORCH[dtype]), dv, 0.7, 1e-5, 0.6)
+    d = a.double()[..., :dv]
+    want = plain.unit_rms(d[:, ::2] - 0.7 * d[:, 1::2], 1e-5) * 0.6
+    close(got, want.reshape(n, heads * dv), dtype)
+    wide = torch.zeros(n, heads * dv + 8, dtype=TORCH[dtype], device="cuda")
+    ops.map_difference(dev(a, TORCH[dtype]), dv, 0.7, 1e-5, 0.6, out=wide[:, 4:4 + heads * dv])
+    assert torch.equal(wide[:, 4:4 + heads * dv], got) and not wide[:, :4].any() and not wide[:, 4 + heads * dv:].any()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,width", [(5, 48), (3, 54), (300, 256), (2, 4096), (9, 8200)])
+def test_two_normed_branches_their_sum_and_the_next_norm(dtype, n, width):
+    from tokamak_b200.csrc import ops
+    gen = torch.Generator().manual_seed(width + n)
+    rnd = _rounded(gen, dtype)
+    x, a, b = torch.randn(n, width, generator=gen), rnd(n, width, std=3.0), rnd(n, width, std=0.2)
+    wa, wb, wn = (torch.randn(width, generator=gen) for _ in range(3))
+    sum_ = x.double() + plain.unit_rms(a.double(), 1e-5) * wa + plain.unit_rms(b.double(), 1e-5) * wb
+    want = plain.unit_rms(sum_, 1e-4) * wn
+    parts = lambda t: dev(torch.stack([0.25 * t, 0.5 * t, 0.25 * t]))
+    for fa, fb in ((lambda t: dev(t, TORCH[dtype]),) * 2, (parts, lambda t: dev(t, TORCH[dtype])), (parts, parts)):
+        resid, out = dev(x), torch.empty(n, width, dtype=TORCH[dtype], device="cuda")
+        ops.branch_pair_norm_add(resid, fa(a), dev(wa), fb(b), dev(wb), 1e-5, dev(wn), out, 1e-4)
+        close(resid, sum_, "float32")
+        close(out, want, dtype)
+        pick = sorted({0, n // 2, n - 1})
+        resid, some = dev(x), torch.empty(len(pick), width, dtype=TORCH[dtype], device="cuda")
+        ops.branch_pair_norm_add(resid, fa(a), dev(wa), fb(b), dev(wb), 1e-5, dev(wn), some, 1e-4, rows=i32(pick))
+        assert torch.equal(resid, dev(x)) and torch.equal(some, out[pick])
+
+
+def _marked(gen, dtype, T, width, marks, queries):
+    """Rows whose channels 0 and 2 mark keys and channel 1 marks queries, and a second, unmarked request."""
+    rnd = _rounded(gen, dtype)
+    seqs = [rnd(T, width, std=0.5), rnd(77, width, std=0.5)]
+    for s in seqs:
+        s[:, :3] = 0.0
+    for channel, at in marks:
+        seqs[0][at, channel] = 8.0
+    seqs[0][queries, 1] = 8.0
+    return seqs
+
+
+def _edges(keys, window, page, T):
+    """Positions around both edges of the window behind every marked key, at page borders, and the last."""
+    at = {4 * page - 1, 4 * page, T - 1}
+    for k in keys:
+        at |= {k + 1, k + window - 2, k + window - 1, k + window, k + window + 1}
+    return sorted(p for p in at if max(keys) < p < T)
+
+
+def _attention_runs(part, seqs, dtype, page, rows, window, heads):
+    """The mixer over a cache of its own: whole prompts, portions down to two tokens beside another request, and
+    the marked stretch token by token; pages in a random order, stale values in those not yet written."""
+    from tokamak_b200.cache.device import KVView
+    T, T2 = len(seqs[0]), len(seqs[1])
+    gen = torch.Generator().manual_seed(T)
+    need = part.cache_need()
+    order, pages = torch.randperm(96, generator=gen).int(), -(-T // page)
+    table = torch.full((4, 60), -1, dtype=torch.int32)
+    table[2, :pages], table[0, :-(-T2 // page)] = order[:pages], order[pages:pages - (-T2 // page)]
+    cuts = [[[T], [T2]], [[7, 2, 30, 2, 64, 3, 2, T - 110], [2, 40, 0, 2, 2, T2 - 46]],
+            [[16] + [1] * (T - 16), [40, 0, 1, 2] + [1] * (T2 - 43)]]
+    width = seqs[0].shape[1]
+    for cut in cuts:
+        k = torch.full((96, need.n_kv_heads, page, need.head_dim), float("nan"), dtype=TORCH[dtype], device="cuda")
+        v = torch.full((96, need.n_kv_heads, page, need.value_dim), float("nan"), dtype=TORCH[dtype], device="cuda")
+        view = KVView(k, v, dev(table), page, window)
+        yield run_in_steps(seqs, [2, 0], cut, lambda x, step: torch.as_tensor(rows(part, dev(x, TORCH[dtype]), step, view)).float(),
+                           heads)
+
+
+def _sum(y, n):
+    return y.float().sum(0) if y.dim() == 3 else y.float()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,d,dv,window,page,dims,scaling", [
+    (3, 1, 10, 14, 9, 4, 6, {"factor": 3.0, "low": 1.0, "high": 4.0, "original": 60}),
+    (4, 2, 32, 64, 40, 16, 32, {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 512}),
+    (4, 4, 16, 20, 17, 16, 12, None), (6, 2, 64, 128, 64, 32, 64, {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 64}),
+    (2, 1, 30, 100, 1, 16, 0, None), (2, 2, 70, 24, 33, 8, 40, None), (16, 2, 24, 40, 300, 16, 24, None)])
+def test_differential_attention_with_keys_that_stand_out_at_the_windows_edges(dtype, H, G, d, dv, window, page, dims, scaling):
+    """A marked key of its own for either map, and marked queries around the two edges of each one's window: the
+    marked pair's score beats every other, so that a key that one map loses or sees too long moves the row by its
+    whole spread (which is checked in the oracle)."""
+    from tokamak_b200.parts.base import MIXERS
+    from tokamak_b200.parts.differential import DifferentialAttentionSpec
+    from tokamak_b200.parts.position import NoPositionSpec, RopeHalvesSpec, WaveScaling
+    gen = torch.Generator().manual_seed(H * 100 + d)
+    rnd = _rounded(gen, dtype)
+    width, T, eps, diff, base = 72, 150, 1e-5, 0.4, 1e5
+    w = {"q": rnd(2 * H * d, width, std=0.1), "k": rnd(2 * G * d, width, std=0.1), "v": rnd(G * dv, width, std=0.3),
+         "o": rnd(width, H * dv, std=0.2)}
+    for name in ("lq1", "lk1", "lq2", "lk2"):
+        w[name] = 0.4 * torch.randn(d, generator=gen) / d ** 0.25
+    w["q"][:, 1], w["k"][:, 0], w["k"][:, 2] = 0.0, 0.0, 0.0
+    w["q"][d - 1::d, 1] = 1.0                                # the piece's last element: unrotated, or turned slowest
+    for g in range(G):
+        w["k"][2 * g * d + d - 1, 0] = 1.0                   # the first map's key
+        w["k"][(2 * g + 1) * d + d - 1, 2] = 1.0             # the second map's
+    marks = [(0, 19), (2, 24)]
+    queries = _edges([19, 24], window, page, T)
+    seqs = _marked(gen, dtype, T, width, marks, queries)
+    m = {"heads": H, "kv_heads": G, "dim": d, "vdim": dv, "scale": 0.45, "diff": diff, "mask": {"size": window},
+         "rot": {"base": base, "dims": dims, "scaling": scaling}}
+    wd = _doubles(w)
+    want = [plain.differential_attention(s.double(), wd, m, eps, torch.arange(len(s))) for s in seqs]
+    for at, other in [(k + window - 1, window - 1) for k in (19, 24)] + [(k + window, window + 1) for k in (19, 24)]:
+        if at in queries and other > 0:          # a window that is one token off would show
+            off = plain.differential_attention(seqs[0].double(), wd, {**m, "mask": {"size": other}}, eps, torch.arange(T))
+            assert (off[at] - want[0][at]).abs().max() > 0.3 * want[0].std(), (at, other)
+    pos = NoPositionSpec() if dims == 0 else RopeHalvesSpec(dims, base, scaling=None if scaling is None else WaveScaling(**scaling))
+    part = _part(MIXERS, DifferentialAttentionSpec(hidden_size=width, num_heads=H, num_kv_heads=G, head_dim=d, v_head_dim=dv,
+                                                   softmax_scale=0.45, position=pos, diff=diff, norm_eps=eps, window=window), w, dtype)
+    assert abs(part.map_weight - float(plain.map_weight(wd, diff))) < 1e-6
+    rows = lambda p, x, step, view: _sum(p.forward(x, step, view), x.shape[0])
+    for got in _attention_runs(part, seqs, dtype, page, rows, window, 2 * H):
+        for g, ref in zip(got, want):
+            close(g, ref, dtype, scale=3.0 if dtype == "float32" else 4.0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,d,dv,window,page,dims,scaling", [
+    (4, 2, 12, 20, 17, 4, 8, {"factor": 4.0, "original": 40, "fast": 8.0, "slow": 1.0}),
+    (4, 1, 64, 64, 40, 16, 64, {"factor": 4.0, "original": 512, "fast": 32.0, "slow": 1.0}),
+    (8, 2, 96, 80, 64, 16, 48, {"factor": 16.0, "original": 128, "fast": 32.0, "slow": 1.0}),
+    (3, 3, 18, 6, 1, 8, 18, None), (2, 2, 40, 128, 33, 32, 40, None), (2, 1, 140, 24, 300, 16, 0, None)])
+def test_attention_with_a_norm_behind_the_rotation_and_sinks(dtype, H, G, d, dv, window, page, dims, scaling):
+    """As above, for queries and keys that are divided by their root mean square after a rotation that also changes
+    their length, and a sink in the denominator."""
+    from tokamak_b200.parts.attention import GatedAttentionSpec
+    from tokamak_b200.parts.base import MIXERS
+    from tokamak_b200.parts.position import NoPositionSpec, RopeHalvesSpec, YarnScaling
+    gen = torch.Generator().manual_seed(H * 100 + d)
+    rnd = _rounded(gen, dtype)
+    width, T, eps, base, scale = 72, 150, 1e-5, 1e6, 18.0 / d
+    w = {"q": rnd(H * d, width, std=0.15), "k": rnd(G * d, width, std=0.15), "v": rnd(G * dv, width, std=0.3),
+         "o": rnd(width, H * dv, std=0.2), "sink": 3.0 + 2.0 * torch.randn(H, generator=gen)}
+    w["q"][:, 1], w["k"][:, 0] = 0.0, 0.0
+    w["q"][d - 1::d, 1] = 4.0
+    w["k"][d - 1::d, 0] = 4.0
+    queries = _edges([19], window, page, T)
+    seqs = _marked(gen, dtype, T, width, [(0, 19)], queries)
+    m = {"heads": H, "kv_heads": G, "dim": d, "vdim": dv, "scale": scale, "mask": {"size": window},
+         "rot": {"base": base, "dims": dims, "scaling": scaling}}
+    wd = _doubles(w)
+    want = [plain.sink_attention(s.double(), wd, m, eps, torch.arange(len(s))) for s in seqs]
+    for at, other in ((19 + window - 1, window - 1), (19 + window, window + 1)):
+        if at in queries and other > 0:
+            off = plain.sink_attention(seqs[0].double(), wd, {**m, "mask": {"size": other}}, eps, torch.arange(T))
+            assert (off[at] - want[0][at]).abs().max() > 0.3 * want[0].std(), (at, other)
+    no_sink = plain.sink_attention(seqs[0].double(), {**wd, "sink": wd["sink"] - 1e9}, m, eps, torch.arange(T))
+    assert (no_sink - want[0]).abs().max() > 0.3 * want[0].std()
+    pos = NoPositionSpec() if dims == 0 else RopeHalvesSpec(dims, base, scaling=None if scaling is None else YarnScaling(**scaling))
+    part = _part(MIXERS, GatedAttentionSpec(hidden_size=width, num_heads=H, num_kv_heads=G, head_dim=d, v_head_dim=dv,
+                                            softmax_scale=scale, position=pos, head_norm_eps=eps, head_norm_weight=False,
+                                            norm_after=True, sinks=True, window=window, pad_rows=True), w, dtype)
+    rows = lambda p, x, step, view: _sum(p.forward(x, step, view), x.shape[0])
+    for got in _attention_runs(part, seqs, dtype, page, rows, window, H):
+        for g, ref in zip(got, want):
+            close(g, ref, dtype, scale=3.0 if dtype == "float32" else 4.0)
+
+
+# ======================================================================= the delta rule with channel decays
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,parts,factors", [(3, 2, [(24, 40), (8, 130)]), (1, 1, [(128, 512), (128, 512)]), (70, 0, [(8, 9)]),
+                                             (64, 3, [(48, 64), (16, 200)]), (9, 0, [(256, 33), (40, 77)])])
+def test_second_halves_of_low_rank_projections(dtype, n, parts, factors):
+    from tokamak_b200.csrc import ops
+    gen = torch.Generator().manual_seed(n)
+    rnd = _rounded(gen, dtype)
+    ranks = [r for r, _ in factors]
+    off = [12 + sum(ranks[:i]) for i in range(len(ranks))]
+    x = rnd(n, 20 + sum(ranks))
+    ws = [rnd(c, r, std=r ** -0.5) for r, c in factors]
+    proj = dev(torch.stack([x / parts] * parts)) if parts else dev(x, TORCH[dtype])
+    got = ops.low_rank(proj, TORCH[dtype], [(o, dev(w, TORCH[dtype])) for o, w in zip(off, ws)])
+    for o, w, g in zip(off, ws, got):
+        assert g.dtype == torch.float32
+        close(g, x[:, o:o + w.shape[1]].double() @ w.double().T, dtype, scale=0.5 if dtype == "bfloat16" else 1.0)
+
+
+CUTS = [[5, 1, 1, 0, 2, 7, 1, 40, 2], [1, 1, 3, 9, 0, 2, 0, 3, 30], [16, 1, 0, 0, 1, 1, 2, 9]]    # the second step is single tokens only
+SLOTS = [2, 0, 3]
+
+
+def _delta_weights(gen, dtype, width, H, G, dk, dv, taps, ra, rg):
+    rnd = _rounded(gen, dtype)
+    s = 1.5 / width ** 0.5
+    w = {"q": rnd(G * dk, width, std=s), "k": rnd(G * dk, width, std=s), "v": rnd(H * dv, width, std=s),
+         "b": rnd(H, width, std=2 * s), "A_log": 0.5 * torch.randn(H, generator=gen),
+         "norm": 1 + 0.3 * torch.randn(dv, generator=gen), "dt_bias": torch.randn(H * dk, generator=gen) - 2.0,
+         "a1": rnd(ra, width, std=s), "a2": rnd(H * dk, ra, std=1.5 / ra ** 0.5), "g1": rnd(rg, width, std=s),
+         "g2": rnd(H * dv, rg, std=1.5 / rg ** 0.5), "o": rnd(width, H * dv, std=(H * dv) ** -0.5)}
+    for n, c in (("q", G * dk), ("k", G * dk), ("v", H * dv)):
+        w[n + ".conv"] = 0.6 * torch.randn(c, taps, generator=gen)
+    return w
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dk,dv,taps,ra,rg", [(4, 2, 12, 10, 3, 5, 11), (3, 1, 7, 9, 1, 8, 3), (2, 2, 64, 64, 4, 24, 24),
+                                                  (4, 4, 130, 33, 2, 16, 40), (2, 1, 256, 20, 6, 7, 8), (8, 4, 128, 128, 4, 128, 128)])
+def test_delta_rule_with_a_decay_per_channel(dtype, H, G, dk, dv, taps, ra, rg):
+    """The mixer cut into steps beside other requests (down to single tokens, with a step of single tokens only, and
+    with pauses), in slots that held another request's state before; and a portion of many tokens."""
+    from tokamak_b200.parts.base import MIXERS
+    from tokamak_b200.parts.delta import GatedDeltaSpec
+    gen = torch.Generator().manual_seed(H * dk + dv)
+    width, eps = 96, 1e-5
+    w = _delta_weights(gen, dtype, width, H, G, dk, dv, taps, ra, rg)
+    part = _part(MIXERS, GatedDeltaSpec(hidden_size=width, num_heads=H, num_kv_heads=G, key_dim=dk, value_dim=dv, conv_taps=taps,
+                                        norm_eps=eps, decay_rank=ra, gate_rank=rg, gate="sigmoid"), w, dtype)
+    m = {"heads": H, "kv_heads": G, "dim": dk, "vdim": dv}
+    rnd = _rounded(gen, dtype)
+    seqs = [rnd(sum(c), width) for c in CUTS]
+    wd = _doubles(w)
+    ROUND = plain.no_round if dtype == "float32" else plain.bf16_round
+    want = [plain.delta_mixer(s.double(), wd, m, eps, ROUND) for s in seqs]
+    records = torch.zeros(4, part.record_floats, device="cuda")
+    view = SimpleNamespace(records=records)
+    fn = lambda x, step: _sum(part.forward(dev(x, TORCH[dtype]), step, view), x.shape[0])
+    tol = 4.0 if dtype == "float32" else 3.0
+    for _ in range(2):
+        records[SLOTS] = 0.0                    # what the cache does when it hands a slot out
+        records[1] = float("nan")               # nobody's slot
+        for g, ref in zip(run_in_steps(seqs, SLOTS, CUTS, fn), want):
+            close(g, ref, dtype, scale=tol)
+    assert records[1].isnan().all()
+    long = rnd(130, width)
+    records[1] = 0.0
+    got = run_in_steps([long], [1], [[80, 2, 48]], fn)[0]
+    close(got, plain.delta_mixer(long.double(), wd, m, eps, ROUND), dtype, scale=tol)
+
+
+def test_channel_decays_each_act_on_their_own_row():
+    """One written key channel per token and decays of exactly 0, 1/2 and 1: what is read back names the row."""
+    from tokamak_b200.csrc import ops
+    dk, dv, H = 8, 5, 2
+    q, k = torch.zeros(4, H, dk), torch.zeros(4, H, dk)
+    v = torch.randn(4, H, dv, generator=torch.Generator().manual_seed(0))
+    k[0, :, 3] = 1.0
+    k[1, :, 5] = 1.0
+    q[2, :, 3], q[2, :, 5] = 1.0, 10.0
+    q[3, :, 3], q[3, :, 5] = 1.0, 10.0
+    g = torch.ones(4, H, dk)
+    g[2, :, 3] = 0.5
+    g[3, 0, 5], g[3, 1, 3] = 0.0, 0.0
+    beta = torch.ones(4, H)
+    step = fake_step([4], [0], [0])
+    rec = torch.zeros(1, H * dk * dv, device="cuda")
+    o = ops.delta_scan(dev(q), dev(k), dev(v), dev(beta), dev(g), rec, step.req_q_start, step.req_q_len, step.req_slot, step.err).cpu()
+    # token 2 and 3 write nothing (k = 0) and read rows 3 and 5
+    assert torch.allclose(o[2], 0.5 * v[0] + 10.0 * v[1]) and torch.allclose(o[3, 0], 0.5 * v[0, 0]) and torch.allclose(o[3, 1], 10.0 * v[1, 1])
+    ref, S = plain.delta_recurrence(*(t.double() for t in (q, k, v, beta, g)))
+    close(o, ref, "float32")
+    close(rec.view(H, dk, dv), S, "float32")
