@@ -456,3 +456,329 @@ def test_channel_decays_each_act_on_their_own_row():
     ref, S = plain.delta_recurrence(*(t.double() for t in (q, k, v, beta, g)))
     close(o, ref, "float32")
     close(rec.view(H, dk, dv), S, "float32")
+
+
+# ======================================================================= experts
+
+@pytest.mark.parametrize("experts,identity,top,count,keep,shared", [
+    (6, 2, 3, 4, 2, 1), (12, 4, 4, 4, 3, 0), (9, 0, 2, 3, 1, 2), (5, 1, 6, 1, 1, 1), (1, 1, 1, 2, 1, 0), (60, 68, 8, 16, 5, 3), (3, 300, 7, 3, 3, 1)])
+def test_router_over_all_outputs_with_groups_identity_and_shared_experts(experts, identity, top, count, keep, shared):
+    """The chosen experts and weights of every token, tokens whose best group holds identity experts only, negative
+    choice scores, the layout of the pairs and the pairs that have no row."""
+    from tokamak_b200.csrc import ops
+    gen = torch.Generator().manual_seed(experts + identity)
+    n, width, total = 500, 40, experts + identity
+    h = torch.randn(n, width, generator=gen)
+    w = {"router": 0.5 * torch.randn(total, width, generator=gen), "correction": 0.2 * torch.randn(total, generator=gen) - 1.0}
+    sg = torch.randn(1, width, generator=gen)
+    chosen, weights, margin = plain.route(h.double(), _doubles(w), {"experts": experts, "identity": identity, "top": top,
+                                                                    "groups": {"count": count, "keep": keep}})
+    router = torch.cat([w["router"], sg]) if shared else w["router"]
+    r = ops.moe_route(dev(h), dev(router), dev(w["correction"]), top=top, n_groups=count, keep=keep, padded=True,
+                      kind="softmax_all", group_score="best", normalize=True, identity=identity, shared=shared)
+    got, gw = r.chosen.cpu().long(), r.weights.cpu().double()
+    clear = margin > 1e-6
+    assert clear.float().mean() > 0.9
+    is_id = chosen >= experts
+    assert torch.equal(got[clear, :top], chosen.masked_fill(is_id, -1)[clear])
+    assert (gw[:, :top] - weights.masked_fill(is_id, 0.0))[clear].abs().max() < 1e-5
+    if identity:
+        own = (weights * is_id).sum(-1)
+        assert (r.identity_weight.cpu()[:, 0].double() - own)[clear].abs().max() < 1e-5
+    if shared:
+        gate = torch.sigmoid(h.double() @ sg.double().T)
+        assert torch.equal(got[:, top:], torch.arange(experts, experts + shared).expand(n, shared))
+        assert (gw[:, top:] - gate).abs().max() < 1e-5
+    # the layout: every pair with a row has one of its own, in a tile of its expert
+    pair_row, tile = r.pair_row.cpu(), r.tile_expert.cpu()
+    flat = got.reshape(-1)
+    assert torch.equal(pair_row >= 0, flat >= 0)
+    rows = pair_row[flat >= 0].long()
+    assert len(set(rows.tolist())) == len(rows) and torch.equal(tile[rows // ops.moe_pad_rows()].long(), flat[flat >= 0])
+    listed = r.order.cpu()[:len(rows)].long()
+    assert torch.equal(listed.sort().values, (flat >= 0).nonzero()[:, 0]) and (flat[listed].diff() >= 0).all()
+
+
+def _moe_weights(gen, dtype, width, ff, experts, identity, shared):
+    rnd = _rounded(gen, dtype)
+    s = 1.5 / width ** 0.5
+    w = {"router": 3 * rnd(experts + identity, width, std=s), "correction": 0.05 * torch.randn(experts + identity, generator=gen)}
+    names = [(f"e{e}.", ff) for e in range(experts)] + ([("shared.", shared)] if shared else [])
+    for p, f in names:
+        w[p + "gate"], w[p + "up"] = rnd(f, width, std=s), rnd(f, width, std=s)
+        w[p + "down"] = rnd(width, f, std=1.5 / f ** 0.5)
+    if shared:
+        w["shared.sg"] = rnd(1, width, std=s)
+    return w
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,width,ff,experts,identity,top,count,keep,shared", [
+    (70, 48, 40, 6, 2, 3, 4, 2, 24), (1, 64, 64, 4, 4, 2, 2, 1, 64), (2, 128, 96, 7, 1, 2, 4, 3, 200), (300, 54, 30, 5, 1, 2, 3, 2, 70),
+    (900, 136, 64, 12, 4, 4, 4, 3, 128), (5, 64, 128, 8, 0, 2, 1, 1, None), (40, 96, 100, 3, 3, 5, 2, 2, None)])
+def test_experts_with_identity_and_shared_ones_through_the_feed_forward(dtype, n, width, ff, experts, identity, top, count, keep, shared):
+    from tokamak_b200.parts.base import FEED_FORWARDS, SumBranch
+    from tokamak_b200.parts.feedforward import MoESpec
+    gen = torch.Generator().manual_seed(n + ff)
+    w = _moe_weights(gen, dtype, width, ff, experts, identity, shared)
+    h = _rounded(gen, dtype)(n, width)
+    mlp = {"router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": count, "keep": keep}},
+           "shared": None if shared is None else {"ff": shared}}
+    margins = []
+    want = plain.mixture(h.double(), _doubles(w), mlp, plain.no_round, margins)
+    part = _part(FEED_FORWARDS, MoESpec(hidden_size=width, intermediate_size=ff, num_experts=experts, top=top, num_groups=count,
+                                        keep_groups=keep, router="softmax_all", normalize=True, group_score="best",
+                                        identity=identity, shared_size=shared, pad_inner=True), w, dtype)
+    if dtype == "bfloat16" and width % 8 == 0:
+        assert part.w_first is not None                 # the tensor cores' grouped product, or the small steps' kernel
+    step = fake_step([n], [0], [0])
+    x = dev(h, TORCH[dtype])
+    clear = margins[0] > 1e-5
+    got = part.forward(x, step)[0]
+    close(got[dev(clear)], want[clear], dtype, scale=2.0)
+    assert got.isfinite().all() and step.err.tolist()[0] == 0
+    # the terms in front of their sum, joined by the kernel of the next norm beside another branch
+    terms = part.forward(x, step, combine=False)
+    terms = terms if isinstance(terms, tuple) else (terms,)
+    assert len(terms) == 1 + (identity > 0)
+    from tokamak_b200.csrc import ops
+    resid = torch.randn(n, width, generator=gen)
+    a = _rounded(gen, dtype)(n, width)
+    out, stream = torch.empty(n, width, dtype=TORCH[dtype], device="cuda"), dev(resid)
+    ops.sum_rmsnorm(stream, (dev(a, TORCH[dtype]), *terms), out, torch.ones(width, device="cuda"), 1e-5)
+    sum_ = resid.double() + a.double() + want
+    close(stream[dev(clear)], sum_[clear], dtype, scale=2.0)
+    settled = dev(resid)
+    SumBranch((dev(a, TORCH[dtype]), *terms)).settle(settled)
+    assert (settled - stream).abs().max() < 1e-4
+    # the result of a token does not depend on the others in the step
+    if dtype == "float32":
+        pick = torch.arange(0, n, 7)
+        assert (part.forward(x[dev(pick)].contiguous(), fake_step([len(pick)], [0], [0]))[0] - got[dev(pick)]).abs().max() < 1e-6
+
+
+# ======================================================================= whole models
+
+LENGTHS = {"XA": [5, 17, 33, 70, 130, 96, 41, 128], "XB": [1, 7, 31, 64, 100, 143, 52, 90],
+           "XC": [3, 40, 77, 150, 64, 110, 25, 95], "XD": [2, 66, 129, 20, 90, 151, 47, 80]}
+TAGS = ["XA", "XB", "XC", "XD"]
+
+
+def requests_for(tag):
+    vocab = sc.ALL[tag][0]["vocab"]
+    return {f"r{i}": random_tokens(vocab, n, seed=100 * i + n) for i, n in enumerate(LENGTHS[tag])}
+
+
+def make_core(tag, dtype, max_tokens, max_live=4):
+    from tokamak_b200.engine.replay import build_core
+    return build_core(folder_of(tag, dtype), dtype, max_tokens, page_size=sc.ALL[tag][2], max_live=max_live)
+
+
+def replay(tag, dtype, builder, max_tokens, poison=False, max_live=4, **kw):
+    from tokamak_b200.engine.replay import run_step
+    reqs = requests_for(tag)
+    if builder is traces.mixed:
+        kw.update(max_tokens=max_tokens, max_live=max_live)
+    records, rows = builder(reqs, **kw)
+    core = make_core(tag, dtype, max_tokens, max_live)
+    results = {}
+    for rec in records:
+        if poison:
+            core.cache.poison_free_pages()
+            core.cache.poison_free_state()
+        out = run_step(core, rec)
+        if out is not None:
+            results[rec["step"]] = out
+        core.manager.check_invariants()
+    assert not core.manager.live_requests()
+    assert all(g.num_free == g.num_pages for g in core.manager.kv_groups)
+    n = check_rows(results, rows, reqs, folder_of(tag, dtype), dtype, f"{tag}/{dtype}")
+    assert n == sum(len(v) for v in rows.values())
+    return core
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("tag", TAGS)
+def test_whole_prompts(tag, dtype):
+    replay(tag, dtype, traces.whole, max_tokens=192)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("tag", TAGS)
+def test_tail_decoded_one_by_one_across_every_window(tag, dtype):
+    replay(tag, dtype, traces.tail_one_by_one, max_tokens=192, tail=70)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("tag", TAGS)
+def test_portions_of_changing_size(tag, dtype):
+    replay(tag, dtype, traces.portions, max_tokens=192)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("tag", TAGS)
+def test_mixed_batches_with_pages_and_slots_used_again(tag, dtype):
+    replay(tag, dtype, traces.mixed, max_tokens=384, poison=True, seed=7)
+    assert sum(LENGTHS[tag]) > 384
+
+
+@pytest.mark.parametrize("seed", [1, 2])
+@pytest.mark.parametrize("tag,dtype", [("XA", "float32"), ("XB", "bfloat16"), ("XC", "bfloat16"), ("XD", "float32")])
+def test_mixed_batches_in_other_orders_with_two_slots(tag, dtype, seed):
+    replay(tag, dtype, traces.mixed, max_tokens=320, poison=True, seed=seed, max_live=2)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_first_tokens_and_long_decode(dtype):
+    """Positions 0, 1, 2 one by one, then 220 more decoded one by one: over many pages that windows give back on
+    the way, the states carried through every step."""
+    from tokamak_b200.engine.replay import run_trace
+    tag = "XA"
+    reqs = {"long": random_tokens(sc.ALL[tag][0]["vocab"], 224, seed=5)}
+    records, rows = traces.tail_one_by_one(reqs, tail=223)
+    results = run_trace(make_core(tag, dtype, 256), records)
+    check_rows(results, rows, reqs, folder_of(tag, dtype), dtype, f"long/{dtype}")
+
+
+def test_same_logits_however_cut_float32():
+    from tokamak_b200.engine.replay import run_trace
+    tag = "XB"
+    reqs = requests_for(tag)
+    got = {}
+    for name, builder in (("whole", traces.whole), ("portions", traces.portions)):
+        records, rows = builder(reqs)
+        res = run_trace(make_core(tag, "float32", 192), records)
+        got[name] = {rp: res[s][i] for s in rows for i, rp in enumerate(rows[s])}
+    for rp, a in got["whole"].items():
+        b = got["portions"][rp]
+        assert np.abs(a - b).max() <= 2e-5 * max(1.0, np.abs(a).max()), rp
+
+
+@pytest.mark.parametrize("tag", TAGS)
+def test_residual_stream_after_every_layer_run_float32(tag):
+    """Layer run by layer run (a looped layer counts every time): the stream with what the block leaves pending
+    added, against the plain implementation."""
+    from tokamak_b200.engine.step import StepEntry
+    from tokamak_b200.parts.base import NormedSum, SumBranch, sum_parts
+    core = make_core(tag, "float32", 64)
+    caught = []
+
+    def joined(resid, pending):
+        u = resid.double()
+        if isinstance(pending, SumBranch):
+            v = torch.zeros_like(resid)
+            pending.settle(v)
+            return u + v.double()
+        if isinstance(pending, NormedSum):
+            for b in (pending.first, pending.second):
+                u = u + plain.unit_rms(sum_parts(b.x).double(), b.eps) * b.weight.double()
+            return u
+        return u + sum_parts(pending).double()
+
+    for block in core.model.blocks.values():
+        def wrapped(resid, pending, step, view, next_norm=None, fwd=block.forward):
+            r, p = fwd(resid, pending, step, view)
+            caught.append(joined(r, p).cpu())
+            return r, p
+        block.forward = wrapped
+    toks = random_tokens(sc.ALL[tag][0]["vocab"], 40, seed=9)
+    core.step.run([StepEntry("a", toks, [39])])
+    cfg, w = plain.load_folder(folder_of(tag, "float32"))
+    want = []
+    plain.forward(cfg, w, toks, layers_out=want)
+    assert len(caught) == len(want) == len(core.model.spec.schedule)
+    for i, got in enumerate(caught):
+        err = (got - want[i]).abs().max().item()
+        assert err <= 2e-4 * max(1.0, want[i].abs().max().item()), f"layer run {i} is off by {err:.3e}"
+
+
+@pytest.mark.parametrize("tag", ["XA", "XB"])
+def test_greedy_generation_through_the_entry_point_float32(tag):
+    """LLM.generate with its scheduler: prompts in portions beside decoding requests, fewer slots
+    than requests, a pool that is used again; the tokens are the plain implementation's."""
+    from tokamak_b200 import LLM, SamplingParams
+    folder = folder_of(tag, "float32")
+    llm = LLM(folder, dtype="float32", block_size=sc.ALL[tag][2], max_seq_len=128, kv_pool_tokens=256,
+              prefill_chunk=24, max_num_batched_tokens=40, max_batch_size=3)
+    vocab = sc.ALL[tag][0]["vocab"]
+    prompts = [random_tokens(vocab, n, seed=7 * n + 1) for n in (5, 33, 1, 61, 18)]
+    outs = llm.generate(prompt_token_ids=prompts, sampling_params=SamplingParams(temperature=0.0, max_new_tokens=10))
+    assert llm.last_stats["mixed_steps"] > 0
+    cfg, w = plain.load_folder(folder)
+    for p, o in zip(prompts, outs):
+        assert o.output_token_ids == plain.greedy_generate(cfg, w, p, 10), len(p)
+
+
+def test_preemption_is_invisible_in_greedy_tokens_float32():
+    """A pool so small that requests are evicted and recomputed: states start over with the request, and the tokens
+    are those of a large pool and of the plain implementation."""
+    from tokamak_b200 import LLM, SamplingParams
+    tag = "XC"                                   # windows of 33 to 80: the pool of the longest runs out
+    folder = folder_of(tag, "float32")
+    prompts = [random_tokens(sc.ALL[tag][0]["vocab"], n, seed=3 * n) for n in (40, 55, 48, 60)]
+    params = SamplingParams(temperature=0.0, max_new_tokens=30)
+    got = {}
+    for pool in (1024, 192):
+        llm = LLM(folder, dtype="float32", block_size=8, max_seq_len=96, kv_pool_tokens=pool, max_batch_size=4)
+        got[pool] = [o.output_token_ids for o in llm.generate(prompt_token_ids=prompts, sampling_params=params)]
+        assert (llm.last_stats["preemptions"] > 0) == (pool == 192)
+    assert got[192] == got[1024]
+    cfg, w = plain.load_folder(folder)
+    assert got[1024][1] == plain.greedy_generate(cfg, w, prompts[1], 30)
+
+
+def test_greedy_generation_bfloat16_with_graphs_picks_top_tokens():
+    """Decode steps replayed from CUDA graphs (every part of the design declares them safe): the tokens are
+    those of the same engine with every step laid out by the host, and nearly the plain implementation's best
+    for their prefix."""
+    from tokamak_b200 import LLM, SamplingParams
+    tag = "XC"
+    folder = folder_of(tag, "bfloat16")
+    llm = LLM(folder, dtype="bfloat16", block_size=sc.ALL[tag][2], max_seq_len=128, max_batch_size=4)
+    assert llm.core.model.graph_safe()
+    prompts = [random_tokens(sc.ALL[tag][0]["vocab"], n, seed=n) for n in (9, 40, 70)]
+    params = SamplingParams(temperature=0.0, max_new_tokens=12)
+    outs = llm.generate(prompt_token_ids=prompts, sampling_params=params)
+    replays = llm.core.step.graph_replays
+    assert replays > 0
+    llm.plain_steps = True
+    slow = llm.generate(prompt_token_ids=prompts, sampling_params=params)
+    assert llm.core.step.graph_replays == replays
+    assert [o.output_token_ids for o in outs] == [o.output_token_ids for o in slow]
+    near = total = 0
+    for p, o in zip(prompts, outs):
+        seq = list(p)
+        for tok in o.output_token_ids:
+            logits = _truth(str(folder), tuple(seq))[0][-1]
+            near += bool(logits[tok] >= logits.max() - 0.1 * logits.std())
+            total += 1
+            seq.append(tok)
+    assert near >= 0.8 * total
+
+
+def test_trace_run_program_on_this_design(tmp_path):
+    tag, dtype = "XD", "float32"
+    reqs = {k: v for k, v in list(requests_for(tag).items())[:4]}
+    records, rows = traces.mixed(reqs, max_tokens=256, seed=3)
+    folder = folder_of(tag, dtype)
+    out = tmp_path / "out"
+    proc = subprocess.run(
+        [sys.executable, str(ROOT / "bin" / "trace_run"), "--model", str(folder), "--dtype", dtype,
+         "--out", str(out), "--max-tokens", "256", "--page-size", "8"],
+        input="".join(json.dumps(r) + "\n" for r in records), text=True, capture_output=True, timeout=600)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert proc.stdout.split() == [w for r in records for w in ("done", str(r["step"]))]
+    vocab = sc.ALL[tag][0]["vocab"]
+    results = {s: np.fromfile(out / f"{s}.f32", dtype="<f4").reshape(-1, vocab) for s in rows}
+    check_rows(results, rows, reqs, folder, dtype, "trace_run")
+
+
+def test_generation_from_the_command_line(capsys):
+    from tokamak_b200.cli import main
+    folder = folder_of("XA", "float32")
+    argv = ["--model", str(folder), "--dtype", "float32", "--prompt-len", "21", "--temperature", "0",
+            "--max-new-tokens", "9", "--ignore-eos", "--block-size", "16", "--max-seq-len", "64", "--kv-pool-tokens", "256"]
+    assert main(argv) == 0
+    first = capsys.readouterr().out
+    assert main(argv) == 0
+    assert capsys.readouterr().out == first and first.strip()
