@@ -1779,12 +1779,227 @@ def puresun_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
     return rows
 
 
+# ------------------------------------------------------------------------------------------------
+# --design sofinex: the Sofinex design beside a Tarivik model of equal layer sizes (the engine's other design with
+# attention beside a recurrent half in one layer and mixtures with groups of experts); its delta rule's kernels
+# beside Logivik's, its attention's beside those of Ketalix
+
+SOFINEX_EXPERTS, SOFINEX_IDENTITY, SOFINEX_TOP, SOFINEX_RANK = 12, 4, 4, 128
+
+
+def sofinex_config(s: dict) -> dict:
+    """Parallel layers (windowed attention with sinks beside the delta rule: width / 128 heads of 128 x 128, low-rank
+    projections of 128) with an ungated feed-forward that holds as many weights as a gated one of width ff, and
+    differential attention layers (two maps of half a head's size over the twin's value heads) with a mixture: 12
+    experts and 4 identity experts of which 4 are used, a shared expert, ff / 4 each.  Two of the layers run twice, so
+    that there are as many layer runs as the twin has layers."""
+    w, d = s["width"], s["dim"]
+    att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "vdim": d, "mask": {"size": s["window"]}}
+    left = dict(att, dim=d, scale=d ** -0.5 * 4.0,
+                rot={"base": 1e6, "dims": d, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    diff = dict(att, dim=d // 2, scale=(d // 2) ** -0.5, diff=0.3,
+                rot={"base": 1e6, "dims": d // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})
+    right = {"heads": w // 128, "kv_heads": w // 128, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": SOFINEX_RANK,
+             "gate_rank": SOFINEX_RANK}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"] // 4}, "shared": {"ff": s["ff"] // 4},
+           "router": {"experts": SOFINEX_EXPERTS, "identity": SOFINEX_IDENTITY, "top": SOFINEX_TOP, "groups": {"count": 4, "keep": 3}}}
+    layers = [{"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": {"kind": "dense", "ff": s["ff"] * 3 // 2}}
+              if i % 2 == 0 else {"type": "attention", "mixer": diff, "mlp": moe} for i in range(s["layers"] - 2)]
+    return {"architecture": "Sofinex", "vocab": s["vocab"], "width": w, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}
+
+
+def sofinex_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> list[dict]:
+    """Every kernel of the design alone, beside the like kernel of the Tarivik, Logivik or Ketalix path at the same
+    shape: time, achieved bytes or flops per second, and the fraction of the measured peak."""
+    import torch
+    from types import SimpleNamespace
+    from tokamak_b200.cache.device import KVView
+    from tokamak_b200.csrc import ops
+    from tokamak_b200.parts.attention import paged_attention
+    from tokamak_b200.parts.base import linear
+    dev = "cuda"
+    gen = torch.Generator(device=dev).manual_seed(0)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    err = torch.zeros(4, dtype=torch.int32, device=dev)
+    hq, hkv, d, page, win, width = s["heads"], s["kv_heads"], s["dim"], 16, s["window"], s["width"]
+    experts, identity, top, ffe, rank = SOFINEX_EXPERTS, SOFINEX_IDENTITY, SOFINEX_TOP, s["ff"] // 4, SOFINEX_RANK
+    bf = lambda *shape: torch.randn(shape, device=dev, generator=gen).bfloat16()
+    f32 = lambda *shape: torch.randn(shape, device=dev, generator=gen)
+    rows = []
+
+    def row(kernel, like, us, us_like, nbytes=0, flops=0.0, like_bytes=0, like_flops=0.0, note=""):
+        r = {"kernel": kernel, "like": like, "us": round(us, 1), "like_us": round(us_like, 1) if us_like else None}
+        for name, t, fl, nb in (("", us, flops, nbytes), ("like_", us_like, like_flops or flops, like_bytes or nbytes)):
+            if not t:
+                continue
+            if fl:
+                r[name + "bf16_frac"] = round(fl / (t * 1e-6) / 1e12 / peaks["bf16_tflops"], 4)
+            elif nb:
+                r[name + "hbm_frac"] = round(nb / (t * 1e-6) / 1e9 / peaks["hbm_gbs"], 4)
+        if note:
+            r["note"] = note
+        rows.append(r)
+
+    sinks, w1 = f32(hq), torch.ones(width, device=dev)
+    router = f32(experts + identity + 1, width) * 0.05
+    corr = f32(experts + identity) * 0.02
+    wgu = ops.moe_stack_gate_up(bf(experts + 1, ffe, width) * width ** -0.5, bf(experts + 1, ffe, width) * width ** -0.5)
+    w_down = bf(experts + 1, width, ffe) * ffe ** -0.5
+    ff = s["ff"] * 3 // 2
+    w_up = bf(ff, width) * width ** -0.5
+    gh, gk, gv = width // 128, 128, 128
+    for name, n, n_req, start in (("prompt", tokens, 1, 0), ("single tokens", batch, batch, ctx - 1)):
+        single, per = n_req > 1, n // n_req
+        t_us = lambda run, **kw: _time_us(run, graph=single, **kw)
+        none = i32([])
+        recs = {}
+        for heads in (hq, 2 * hq):
+            rec, n_parts, n_split = ops.prefill_tc_records([0] if not single else list(range(n)), [per] * n_req, [start + per] * n_req,
+                                                           list(range(n_req)), heads=heads, sms=ops.sm_count(torch.device(dev, 0)))
+            recs[heads] = ops.PrefillItems(torch.from_numpy(rec).to(dev), n_parts, n_split)
+        step = SimpleNamespace(decode_items=i32(list(range(n))) if single else none, prefill_items=none if single else i32(list(range(n))),
+                               prefill_tiles=none, positions=i32([start + i for _ in range(n_req) for i in range(per)]),
+                               tok_req=i32([r for r in range(n_req) for _ in range(per)]), req_q_start=i32([r * per for r in range(n_req)]),
+                               req_q_len=i32([per] * n_req), req_kv_len=i32([start + per] * n_req), req_slot=i32(list(range(n_req))),
+                               err=err, max_q_len=per, n_tokens=n, scratch={}, max_kv_len=start + per, prefill_tc=recs[hq])
+        pages_req = -(-(start + per) // page)
+        table = torch.randperm(n_req * pages_req, device=dev, generator=gen).to(torch.int32).view(n_req, pages_req)
+        kc, vc = bf(n_req * pages_req, hkv, page, d), bf(n_req * pages_req, hkv, page, d)
+        view = KVView(kc, vc, table, page, win)
+        keys = sum(min(start + i + 1, win) for _ in range(n_req) for i in range(per))
+        # ---- attention: one map a head as Ketalix runs it, with a sink, and two maps a head
+        q1, q2 = bf(n, hq, d), bf(n, 2 * hq, d)
+        o1, o2 = torch.empty_like(q1), torch.empty_like(q2)
+
+        def attention(q, o, **kw):
+            step.prefill_tc = recs[q.shape[1]]
+            return t_us(lambda: paged_attention(q, o, view, step, scale=d ** -0.5, window=win, **kw))
+        like = attention(q1, o1, softcap=30.0, sinks=sinks)
+        kv_bytes = 2 * hkv * keys * d * 2
+        kw = lambda maps: (dict(nbytes=kv_bytes + 2 * maps * q1.numel() * 2, like_bytes=kv_bytes + 2 * q1.numel() * 2) if single else
+                           dict(flops=keys * hq * (4.0 * d if maps == 1 else 6.0 * d), like_flops=4.0 * keys * hq * d))
+        row(f"windowed attention with sinks, {name}", f"windowed attention (cap, sink), {name}", attention(q1, o1, sinks=sinks), like, **kw(1))
+        row(f"differential attention (two maps), {name}", f"windowed attention (cap, sink), {name}", attention(q2, o2), like, **kw(2),
+            note="" if single else "the maps' keys fill a row together, so the scores' product runs over twice the elements it needs")
+        # ---- what stands around it
+        freq = lambda dims: (1.0 / (1e6 ** (torch.arange(0, dims, 2, dtype=torch.float32) / dims))).to(dev)
+        rope, rope_half = ops.rope_table(step.positions, freq(d), 1.1), ops.rope_table(step.positions, freq(d // 2))
+        qkv = bf(n, (hq + 2 * hkv) * d)
+        off = dict(q_off=0, k_off=hq * d, v_off=(hq + hkv) * d)
+        pairs = t_us(lambda: ops.qkv_pairs(qkv, q1, kc, vc, step.positions, step.tok_req, step.req_slot, table, rope, err, n_q_heads=hq,
+                                           n_kv_heads=hkv, rotary_dim=d, unit_norm_eps=1e-6, req_q_len=step.req_q_len,
+                                           req_kv_len=step.req_kv_len))
+        nb = 2 * qkv.numel() * 2 + rope.numel() * 4
+        row(f"rotation (halves), norm behind it, page write, {name}", f"pair rotation + unit norm + page write, {name}",
+            t_us(lambda: ops.qkv_heads(qkv, q1, kc, vc, step, table, head_norm_eps=1e-6, norm_after=True, table=rope, rotary_dim=d,
+                                       halves=True, **off)), pairs, nbytes=nb)
+        row(f"rotation and page write for two maps a head, {name}", f"pair rotation + unit norm + page write, {name}",
+            t_us(lambda: ops.qkv_heads(qkv, q2, kc, vc, step, table, table=rope_half, rotary_dim=d // 2, halves=True, maps=2,
+                                       k_dim=d // 2, v_dim=d, **off)), pairs,
+            nbytes=nb + q1.numel() * 2, like_bytes=nb)
+        g_proj = bf(n, hq * d)
+        row(f"difference of the maps, norm, scale, {name}", f"output gate into rows, {name}",
+            t_us(lambda: ops.map_difference(o2, d, 0.4, 1e-6, 0.7)), t_us(lambda: ops.gate_scale(o1.view(n, hq * d), g_proj, 0)),
+            nbytes=3 * n * hq * d * 2)
+        # ---- the delta rule: second halves, inputs, recurrence, output stage
+        ch = gh * gk
+        cols = 3 * ch + 2 * rank + gh
+        proj = bf(n, cols) * 0.5
+        conv, a_log = f32(3 * ch, 4) * 0.5, f32(gh) * 0.5
+        wa, wg = bf(ch, rank) * rank ** -0.5, bf(ch, rank) * rank ** -0.5
+        if single:
+            parts = proj.float().unsqueeze(0).repeat(2, 1, 1) * 0.5
+            halves = lambda: ops.low_rank(parts, torch.bfloat16, [(3 * ch, wa), (3 * ch + rank, wg)])
+            za, zg = (z.unsqueeze(0) for z in halves())
+        else:
+            halves = lambda: (torch.mm(proj[:, 3 * ch:3 * ch + rank], wa.t()), torch.mm(proj[:, 3 * ch + rank:3 * ch + 2 * rank], wg.t()))
+            za, zg = halves()
+        row(f"second halves of the low-rank projections, {name}", None, t_us(halves), 0.0,
+            nbytes=2 * ch * rank * 2 + n * (2 * rank * 2 + 2 * ch * za.element_size()))
+        floats, _ = ops.delta_record_floats(gh, gh, gk, gv, 4)
+        records = torch.zeros(n_req, floats, device=dev)
+        pk = dict(dtype=torch.bfloat16, q_off=0, k_off=ch, v_off=2 * ch, b_off=3 * ch + 2 * rank, a_off=3 * ch, heads=gh, kv_heads=gh,
+                  key_dim=gk, value_dim=gv, unit_eps=1e-6, q_scale=gk ** -0.5)
+        args = (records, step.tok_req, step.req_q_start, step.req_q_len, step.req_slot, err)
+        dt_c, dt_h = f32(ch) - 2.0, f32(gh) - 2.0
+        prep = lambda: ops.delta_prepare(proj, conv, a_log, dt_c, *args, channel_a=za, **pk)
+        prep_h = lambda: ops.delta_prepare(proj, conv, a_log, dt_h, *args, **pk)
+        row(f"delta rule inputs with channel decays, {name}", f"delta rule inputs with one decay a head, {name}", t_us(prep), t_us(prep_h),
+            nbytes=n * ch * (3 * 2 + za.element_size() + 4 * 4), like_bytes=n * ch * (3 * 2 + 3 * 4))
+        x, xh = prep(), prep_h()
+        scan = lambda v: lambda: ops.delta_scan(*v, records, step.req_q_start, step.req_q_len, step.req_slot, err)
+        us, us_h = t_us(scan(x)), t_us(scan(xh))
+        state = 2 * n_req * gh * gk * gv * 4
+        rows.append({"kernel": f"delta rule recurrence with channel decays, {name}", "like": f"delta rule recurrence with one decay a head, {name}",
+                     "us": round(us, 1), "like_us": round(us_h, 1),
+                     "hbm_frac": round((state + n * ch * 5 * 4) / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 4),
+                     "like_hbm_frac": round((state + n * ch * 4 * 4) / (us_h * 1e-6) / 1e9 / peaks["hbm_gbs"], 4),
+                     "fp32_tflops": round(8.0 * n * ch * gv / (us * 1e-6) / 1e12, 2),
+                     "like_fp32_tflops": round(8.0 * n * ch * gv / (us_h * 1e-6) / 1e12, 2)})
+        o = scan(x)()
+        norm = torch.ones(gv, device=dev)
+        row(f"delta rule output norm + sigmoid gate, {name}", f"the same with silu and the gate in the stacked rows, {name}",
+            t_us(lambda: ops.gla_out(o, zg, 0, norm, 1e-6, torch.bfloat16, gate="sigmoid")),
+            t_us(lambda: ops.gla_out(o, proj, 0, norm, 1e-6, torch.bfloat16)),
+            nbytes=n * ch * (4 + zg.element_size() + 2), like_bytes=n * ch * 8)
+        # ---- the two halves' norms, their sum and the next norm
+        resid, normed = f32(n, width), torch.empty(n, width, dtype=torch.bfloat16, device=dev)
+        out_w = bf(width, hq * d) * 0.02
+        a, b = (linear(bf(n, hq * d), out_w, err=err) for _ in range(2))
+        ops.flush_chains()
+        el = a.numel() * a.element_size()
+        row(f"norms of both halves, their sum, residual, input norm, {name}", f"output norm + residual + input norm, {name}",
+            t_us(lambda: ops.branch_pair_norm_add(resid, a, w1, b, w1, 1e-6, w1, normed, 1e-6)),
+            t_us(lambda: ops.branch_norm_add(resid, a, w1, None, 1e-6, w1, normed, 1e-6)),
+            nbytes=n * width * 10 + 2 * el, like_bytes=n * width * 10 + el)
+        # ---- dense feed-forward's first product
+        h = bf(n, width)
+
+        def up(act):
+            if ops.pair_gemm_takes(n, ff, width, fused=True):
+                return lambda: ops.gemm_pair(h, w_up, err, unary=act)
+            splits, stages, cluster = ops.swapped_gemm_plan(ff, width, n)
+            return lambda: ops.gemm_tc_swapped(w_up, h, err, splits, max_stages=stages, cluster=cluster, unary=act)
+        row(f"up product with the exact gelu, {name}", f"up product with relu squared, {name}", t_us(up("gelu")), t_us(up("relu2")),
+            **(dict(nbytes=w_up.numel() * 2) if single else dict(flops=2.0 * n * ff * width)))
+        # ---- the experts
+        rk = dict(top=top, n_groups=4, keep=3, padded=True)
+        mine = lambda: ops.moe_route(h, router, corr, kind="softmax_all", group_score="best", normalize=True, identity=identity,
+                                     shared=1, **rk)
+        row(f"router over all outputs, identity and shared experts, {name}", f"sigmoid router with groups, {name}",
+            _time_us(mine, graph=True), _time_us(lambda: ops.moe_route(h, router[:-1], corr, **rk), graph=True),
+            nbytes=n * width * 2 + router.numel() * 4)
+        routing = mine()
+        plain_r = ops.moe_route(h, router[:experts].contiguous(), None, **rk)
+        small = ops.moe_small_takes(n, top + 1, width, ffe)
+        run = lambda r, wa, wb, small: ((lambda: ops.moe_experts_small(h, r, wa, wb, combine=False)) if small else
+                                        (lambda: ops.moe_experts_tc(h, r, wa, wb, err, combine=False)))
+        chosen = routing.chosen
+        live = int((chosen >= 0).sum())
+        used, used_p = len(set(chosen[chosen >= 0].tolist())), len(set(plain_r.chosen.flatten().tolist()))
+        size = 3 * ffe * width
+        row(f"experts and the shared one, {name}", f"experts (gated), {name}", t_us(run(routing, wgu, w_down, small)),
+            t_us(run(plain_r, wgu[:experts], w_down[:experts], ops.moe_small_takes(n, top, width, ffe))),
+            **(dict(nbytes=2 * used * size, like_bytes=2 * used_p * size) if single else
+               dict(flops=2.0 * live * size, like_flops=2.0 * n * top * size)),
+            note=f"{live} of {n * (top + 1)} pairs have an expert with weights" + (f"; {used} of {experts + 1} are read" if single else ""))
+        y, own = run(routing, wgu, w_down, small)(), ops.WeightedRows(h, routing.identity_weight, None)
+        y_p = run(plain_r, wgu[:experts], w_down[:experts], ops.moe_small_takes(n, top, width, ffe))()
+        row(f"weighted sum of experts + identity rows + residual + input norm, {name}", f"weighted sum of experts + residual + input norm, {name}",
+            t_us(lambda: ops.sum_rmsnorm(resid, (y, own), normed, w1, 1e-6)), t_us(lambda: ops.sum_rmsnorm(resid, (y_p,), normed, w1, 1e-6)),
+            nbytes=n * width * (10 + 2) + live * width * y.y.element_size(), like_bytes=n * width * (10 + top * y_p.y.element_size()))
+    assert err.tolist()[0] == 0, err.tolist()
+    return rows
+
+
 DESIGNS = {
     "ketalix": dict(name="Ketalix", config=ketalix_config, twin=("qwen3_twin", qwen3_twin), kernels=ketalix_kernels),
     "logivik": dict(name="Logivik", config=logivik_config, twin=("ketalix_twin", ketalix_config), kernels=logivik_kernels),
     "tarivik": dict(name="Tarivik", config=tarivik_config, twin=("ketalix_twin", ketalix_config), kernels=tarivik_kernels),
     "pukinex": dict(name="Pukinex", config=pukinex_config, twin=("ketalix_twin", ketalix_config), kernels=pukinex_kernels),
     "puresun": dict(name="Puresun", config=puresun_config, twin=("logivik_latent_twin", logivik_latent_twin), kernels=puresun_kernels),
+    "sofinex": dict(name="Sofinex", config=sofinex_config, twin=("tarivik_twin", tarivik_config), kernels=sofinex_kernels),
 }
 
 
@@ -1894,7 +2109,7 @@ def main() -> int:
                          "own, 14b, 32b)")
     ap.add_argument("--design", default=None, choices=sorted(DESIGNS),
                     help="measure another design instead: its prefill and decode throughput beside the engine's closest "
-                         "other model of equal layer sizes (Ketalix beside Qwen3, Puresun beside Logivik, the rest beside Ketalix), and its kernels "
+                         "other model of equal layer sizes (Ketalix beside Qwen3, Puresun beside Logivik, Sofinex beside Tarivik, the rest beside Ketalix), and its kernels "
                          "alone beside their like kernels (--design-sizes)")
     ap.add_argument("--design-sizes", default="2b", choices=sorted(KETALIX_SIZES))
     ap.add_argument("--num-requests", type=int, default=32)

@@ -306,6 +306,129 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
   }
 }
 
+// The same for pieces of up to 128 elements (sizes, offsets and row lengths multiples of 4, the rotated part in whole
+// fours per half, values of their own): kLanes lanes take a piece, four elements each, so that a warp works on 32 /
+// kLanes pieces, and rotation partners and sums of squares pass between lanes instead of through shared memory.
+template <typename T, int kLanes>
+__global__ void __launch_bounds__(kHeadsWarps * 32) qkv_heads_lanes_kernel(QkvHeadsParams p) {
+  constexpr int kPieces = 32 / kLanes;
+  pdl_trigger();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int first = (blockIdx.y * kHeadsWarps + warp) * kPieces;
+  const int k_heads = p.n_kv_heads * p.maps, heads_total = p.n_q_heads + k_heads + p.n_kv_heads;
+  if (first >= heads_total) return;                    // the whole warp
+  const int t = blockIdx.x;
+  const int h = min(first + lane / kLanes, heads_total - 1);
+  const bool real = first + lane / kLanes < heads_total;
+  const int kind = h < p.n_q_heads ? 0 : h < p.n_q_heads + k_heads ? 1 : 2;       // 0 = q, 1 = k, 2 = v
+  const int head = kind == 0 ? h : kind == 1 ? h - p.n_q_heads : h - p.n_q_heads - k_heads;
+  const int d = kind == 2 ? p.v_dim : p.k_dim;
+  const int c = lane % kLanes, e = 4 * c;
+  const bool live = real && e < d;
+  const int r = p.rope_table != nullptr && kind != 2 ? p.rotary_dim : 0, half = r >> 1;
+  pdl_wait();
+  float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  if (live) {
+    x = stacked_ld4<T>(p.in, (size_t)t * p.in.row_stride + (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + head * d + e);
+  }
+  // the angles of these four elements: four pairs (halves) or two (neighbours)
+  float4 cs0 = make_float4(1.0f, 0.0f, 1.0f, 0.0f), cs1 = cs0;
+  const bool turned = e < r;
+  if (turned) {
+    const float2* tab = p.rope_table + (size_t)t * half;
+    if (p.halves) {
+      const int i = e < half ? e : e - half;
+      cs0 = *reinterpret_cast<const float4*>(tab + i); cs1 = *reinterpret_cast<const float4*>(tab + i + 2);
+    } else {
+      const float2 a = tab[e >> 1], b = tab[(e >> 1) + 1];
+      cs0 = make_float4(a.x, a.y, b.x, b.y);
+    }
+  }
+  const int pos = p.positions[t];
+  bool ok = real;
+  if (pos < 0) { if (lane == 0) set_error(p.err, kErrPosition, t, pos, 0); return; }      // the whole warp
+  const int row_len = kind == 2 ? p.v_row : p.k_row;
+  const int piece = kind == 2 ? 0 : head % p.maps, off = piece * d;
+  const int tail = kind == 2 || piece == p.maps - 1 ? row_len - off : d;
+  T* dst = (T*)p.q_out + ((size_t)t * p.n_q_heads + (kind == 0 ? head : 0)) * row_len;
+  int zero_rows = 0;
+  if (kind != 0) {
+    const int req = p.tok_req[t];
+    const int pidx = pos / p.page_size, slot = pos - pidx * p.page_size;
+    int page = -1;
+    if (req < 0 || req >= p.n_reqs) {
+      if (lane % kLanes == 0) set_error(p.err, kErrRequest, t, req, p.n_reqs);
+    } else {
+      page = pidx < p.max_pages ? p.block_table[(size_t)p.req_slot[req] * p.max_pages + pidx] : -1;
+      if (page < 0 || page >= p.num_pages) { if (lane % kLanes == 0) set_error(p.err, kErrPage, t, pidx, page); page = -1; }
+    }
+    ok = ok && page >= 0;
+    const size_t row = ((size_t)max(page, 0) * p.n_kv_heads + (kind == 1 ? head / p.maps : head)) * p.page_size + slot;
+    dst = (T*)(kind == 1 ? p.k_cache : p.v_cache) + row * row_len;
+    // the request's last token of this step clears the rest of a page that was begun in this step
+    if (ok && p.req_kv_len != nullptr) {
+      const int kv_len = p.req_kv_len[req], q_len = p.req_q_len[req];
+      if (pos == kv_len - 1 && pos - slot >= kv_len - q_len) zero_rows = p.page_size - 1 - slot;
+    }
+  }
+  if (live) {
+    const float* bias = kind == 0 ? p.q_bias : kind == 1 ? p.k_bias : p.v_bias;
+    if (bias != nullptr) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + head * d + e);
+      x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
+    }
+  }
+  auto piece_sum = [&](float v) {
+#pragma unroll
+    for (int o = kLanes / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+  };
+  auto scale4 = [](float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); };
+  const float* w = p.head_norm && kind != 2 ? (kind == 0 ? p.q_norm : p.k_norm) : nullptr;
+  auto norm = [&]() {
+    const float f = rsqrtf(piece_sum((x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w)) / (float)d + p.eps);
+    if (kind == 2) return;
+    x = scale4(x, f);
+    if (w != nullptr && live) {
+      const float4 g = *reinterpret_cast<const float4*>(w + e);
+      x.x *= g.x; x.y *= g.y; x.z *= g.z; x.w *= g.w;
+    }
+  };
+  if (p.head_norm && !p.norm_after) norm();
+  if (p.rope_table != nullptr) {
+    if (p.halves) {
+      const int q4 = half >> 2;
+      const int from = (lane - c) + (e < half ? c + q4 : c - q4);
+      const int src = turned ? from : lane;
+      float4 o;
+      o.x = __shfl_sync(0xffffffffu, x.x, src); o.y = __shfl_sync(0xffffffffu, x.y, src);
+      o.z = __shfl_sync(0xffffffffu, x.z, src); o.w = __shfl_sync(0xffffffffu, x.w, src);
+      if (turned) {
+        const float s = e < half ? -1.0f : 1.0f;
+        x = make_float4(x.x * cs0.x + s * (o.x * cs0.y), x.y * cs0.z + s * (o.y * cs0.w), x.z * cs1.x + s * (o.z * cs1.y),
+                        x.w * cs1.z + s * (o.w * cs1.w));
+      }
+    } else if (turned) {
+      x = make_float4(x.x * cs0.x - x.y * cs0.y, x.y * cs0.x + x.x * cs0.y, x.z * cs0.z - x.w * cs0.w, x.w * cs0.z + x.z * cs0.w);
+    }
+  }
+  if (p.head_norm && p.norm_after) norm();
+  if (kind == 0 && p.temp_every > 0) x = scale4(x, 1.0f + p.temp_coef * logf(floorf((float)(pos + 1) / (float)p.temp_every) + 1.0f));
+  if (!ok) return;
+  const float4 zero4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  if (live) st4<T>(dst + off + e, x);
+  if (kind == 0) {
+    for (int i = e; i < row_len; i += 4 * kLanes) {
+      if (i < off || i >= off + d) st4<T>(dst + i, zero4);
+    }
+    return;
+  }
+  for (int i = d + e; i < tail; i += 4 * kLanes) st4<T>(dst + off + i, zero4);
+  for (int z = 1; z <= zero_rows; ++z) {
+    for (int i = e; i < tail; i += 4 * kLanes) st4<T>(dst + (size_t)z * row_len + off + i, zero4);
+  }
+}
+
 }  // namespace tk
 
 TK_API int tk_qkv_heads(const void* x, const float* parts, int n_parts, long long part_stride, int row_stride,
@@ -344,6 +467,17 @@ TK_API int tk_qkv_heads(const void* x, const float* parts, int n_parts, long lon
   cudaError_t e = cudaSuccess;
   const bool vec = k_dim % 4 == 0 && v_dim % 4 == 0 && k_row % 4 == 0 && v_row % 4 == 0 && row_stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
                    (v_off < 0 || v_off % 4 == 0);
+  const int widest = k_dim > v_dim ? k_dim : v_dim;
+  if (vec && widest <= 128 && v_off >= 0 && (rope_table == nullptr || rotary_dim % (halves ? 8 : 4) == 0) &&
+      ((uintptr_t)rope_table & 15) == 0) {
+    const int lanes = widest <= 32 ? 8 : widest <= 64 ? 16 : 32, per_block = tk::kHeadsWarps * (32 / lanes);
+    const dim3 g((unsigned)n_tokens, (unsigned)((heads_total + per_block - 1) / per_block));
+#define TK_QKV_LANES(L) \
+    TK_DISPATCH_DTYPE(dtype, T, (e = tk::launch(tk::qkv_heads_lanes_kernel<T, L>, g, dim3(tk::kHeadsWarps * 32), 0, stream, p)))
+    if (lanes == 8) { TK_QKV_LANES(8); } else if (lanes == 16) { TK_QKV_LANES(16); } else { TK_QKV_LANES(32); }
+#undef TK_QKV_LANES
+    return (int)e;
+  }
   if (vec) {
     TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::qkv_heads_vec_kernel<T>, grid, dim3(tk::kHeadsWarps * 32), 0, stream, p));
     return (int)e;
