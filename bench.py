@@ -1851,7 +1851,7 @@ def sofinex_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
     gh, gk, gv = width // 128, 128, 128
     for name, n, n_req, start in (("prompt", tokens, 1, 0), ("single tokens", batch, batch, ctx - 1)):
         single, per = n_req > 1, n // n_req
-        t_us = lambda run, **kw: _time_us(run, graph=single, **kw)
+        t_us = lambda run: _time_us(run, graph=single)
         none = i32([])
         recs = {}
         for heads in (hq, 2 * hq):
@@ -1968,7 +1968,7 @@ def sofinex_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
         mine = lambda: ops.moe_route(h, router, corr, kind="softmax_all", group_score="best", normalize=True, identity=identity,
                                      shared=1, **rk)
         row(f"router over all outputs, identity and shared experts, {name}", f"sigmoid router with groups, {name}",
-            _time_us(mine, graph=True), _time_us(lambda: ops.moe_route(h, router[:-1], corr, **rk), graph=True),
+            t_us(mine), t_us(lambda: ops.moe_route(h, router[:-1], corr, **rk)),
             nbytes=n * width * 2 + router.numel() * 4)
         routing = mine()
         plain_r = ops.moe_route(h, router[:experts].contiguous(), None, **rk)

@@ -434,6 +434,45 @@ def test_delta_rule_with_a_decay_per_channel(dtype, H, G, dk, dv, taps, ra, rg):
     close(got, plain.delta_mixer(long.double(), wd, m, eps, ROUND), dtype, scale=tol)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dk,dv,taps", [(4, 2, 12, 20, 3), (3, 3, 130, 33, 2), (2, 1, 64, 200, 4), (2, 2, 7, 9, 6)])
+def test_delta_rule_inputs_in_every_launch_shape(dtype, H, G, dk, dv, taps):
+    """Requests whose tokens begin and end inside the runs of tokens that a warp takes; the same bits and the same
+    tails from every shape, and a step so large that the launcher takes the shape for many tokens itself."""
+    from tokamak_b200.csrc import ops
+    gen = torch.Generator().manual_seed(dk)
+    rnd = _rounded(gen, dtype)
+    lens = [1, 5, 2, 1, 9, 700, 3, 2]
+    n, cols, chans = sum(lens), 2 * G * dk + H * dv + H, 2 * G * dk + H * dv
+    proj, a = dev(rnd(n, cols), TORCH[dtype]), dev(rnd(n, H * dk), TORCH[dtype])
+    conv, a_log, bias = 0.5 * torch.randn(chans, taps, generator=gen), torch.randn(H, generator=gen), torch.randn(H * dk, generator=gen)
+    floats, tail_off = ops.delta_record_floats(H, G, dk, dv, taps)
+    start = torch.randn(9, floats, generator=gen)
+    slots = [3, 8, 1, 0, 5, 2, 7, 4]
+    step = fake_step(lens, slots, [4] * len(lens))
+    kw = dict(dtype=TORCH[dtype], q_off=0, k_off=G * dk, v_off=2 * G * dk, b_off=chans, a_off=0, heads=H, kv_heads=G, key_dim=dk,
+              value_dim=dv, unit_eps=1e-6, q_scale=dk ** -0.5, channel_a=a)
+    got = []
+    for shape in (1, 2, 3, 0):
+        records = dev(start)
+        got.append((*ops.delta_prepare(proj, dev(conv), dev(a_log), dev(bias), records, step.tok_req, step.req_q_start, step.req_q_len,
+                                       step.req_slot, step.err, shape=shape, **kw), records))
+    assert step.err.tolist()[0] == 0
+    for other in got[1:]:
+        assert all(torch.equal(x, y) for x, y in zip(got[0], other))
+    x = proj.cpu().double()
+    at = 0
+    for n_r, slot in zip(lens, slots):          # against the plain functions, continuing from the tails
+        past = start[slot, tail_off:].view(taps - 1, chans).double()
+        y = plain.short_conv(torch.cat([past, x[at:at + n_r, :chans]]), conv.double())[taps - 1:]
+        q = plain.unit_vector(y[:, :G * dk].reshape(n_r, G, dk)) * dk ** -0.5
+        k = plain.unit_vector(y[:, G * dk:2 * G * dk].reshape(n_r, G, dk))
+        g = plain.channel_decay(a[at:at + n_r].cpu().double(), a_log.double(), bias.double())
+        for want, have in zip((q, k, y[:, 2 * G * dk:].reshape(n_r, H, dv), torch.sigmoid(x[at:at + n_r, chans:]), g), got[3]):
+            close(have[at:at + n_r], want, "float32")
+        at += n_r
+
+
 def test_channel_decays_each_act_on_their_own_row():
     """One written key channel per token and decays of exactly 0, 1/2 and 1: what is read back names the row."""
     from tokamak_b200.csrc import ops

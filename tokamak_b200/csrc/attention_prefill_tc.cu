@@ -197,7 +197,6 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
   const int group = p.n_q_heads / p.n_kv_heads;
   const int n_items = p.n_records * p.n_q_heads;       // heads vary fastest: the query heads that share a
                                                        // kv head run at the same time and find its pages in L2
-  pdl_trigger();
   if (threadIdx.x == 0) {
     for (int s = 0; s < kAtStages; ++s) {
       mbar_init(gt_smem_u32(&k_full[s]), 1);
@@ -231,6 +230,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
+  // only now may later kernels begin: none of them can take tensor memory before this block has its own
+  pdl_trigger();
   pdl_wait();     // queries, cache pages and the item list come from earlier kernels and copies
 
   if (warp == 0) {

@@ -164,6 +164,169 @@ __global__ void delta_prepare_kernel(DeltaPrepareParams p) {
   }
 }
 
+// The same for steps of many tokens: a warp takes a head for kPrepTokens tokens in a row, the convolution's window
+// slides through registers (one input load a token and channel), q and k stay in registers until their length is
+// known.  Sums are formed in the order of the kernel above: a position's inputs are the same bits.  kTaps: 2 to 4.
+constexpr int kPrepTokens = 4;
+
+template <typename T, int kTaps>
+__global__ void __launch_bounds__(kDeltaPrepWarps * 32) delta_prepare_rows_kernel(DeltaPrepareParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * kPrepTokens, cnt = min(kPrepTokens, p.n_tokens - t0);
+  const int unit = blockIdx.y * kDeltaPrepWarps + (threadIdx.x >> 5);
+  if (unit >= 2 * p.kv_heads + p.heads) return;
+  const int kind = unit < p.kv_heads ? 0 : unit < 2 * p.kv_heads ? 1 : 2;      // 0 = q, 1 = k, 2 = v
+  const int head = kind == 0 ? unit : kind == 1 ? unit - p.kv_heads : unit - 2 * p.kv_heads;
+  const int d = kind == 2 ? p.dv : p.dk;
+  const int hk = p.kv_heads * p.dk, channels = 2 * hk + p.heads * p.dv;
+  const int chan0 = kind == 0 ? head * p.dk : kind == 1 ? hk + head * p.dk : 2 * hk + head * p.dv;
+  const int col0 = kind == 0 ? p.q_off + head * p.dk : kind == 1 ? p.k_off + head * p.dk : p.v_off + head * p.dv;
+  // the tokens' places among their requests' tokens, and their tails
+  int place[kPrepTokens];
+  const float* tails[kPrepTokens];
+  bool ok[kPrepTokens];
+#pragma unroll
+  for (int i = 0; i < kPrepTokens; ++i) {
+    const int t = t0 + i;
+    place[i] = 0; tails[i] = nullptr; ok[i] = false;
+    if (i >= cnt) continue;
+    const int r = p.tok_req[t];
+    if (r < 0 || r >= p.n_reqs) { if (lane == 0) set_error(p.err, kErrRequest, t, r, p.n_reqs); continue; }
+    const int slot = p.req_slot[r];
+    if (slot < 0 || slot >= p.n_slots) { if (lane == 0) set_error(p.err, kErrRequest, t, slot, p.n_slots); continue; }
+    place[i] = t - p.req_q_start[r];
+    tails[i] = p.state + (size_t)slot * p.rec_stride + p.tail_off;
+    ok[i] = true;
+  }
+  float* dst = kind == 0 ? p.q_out + ((size_t)t0 * p.kv_heads + head) * p.dk
+             : kind == 1 ? p.k_out + ((size_t)t0 * p.kv_heads + head) * p.dk
+                         : p.v_out + ((size_t)t0 * p.heads + head) * p.dv;
+  const size_t dst_stride = kind == 2 ? (size_t)p.heads * p.dv : (size_t)p.kv_heads * p.dk;
+  // The usual run: four tokens of one request with the whole window among this step's rows.  Its loads stand in one
+  // stretch without a branch between them.
+  bool usual = place[0] >= kTaps - 1;
+#pragma unroll
+  for (int i = 0; i < kPrepTokens; ++i) usual = usual && ok[i] && place[i] == place[0] + i;
+  auto usual_channel = [&](int e, float (&y)[kPrepTokens]) {
+    float w[kTaps], x[kPrepTokens + kTaps - 1];
+    const size_t row = (size_t)(t0 - (kTaps - 1)) * p.in.row_stride + col0 + e;
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) w[j] = p.taps[(size_t)(chan0 + e) * kTaps + j];
+#pragma unroll
+    for (int j = 0; j < kPrepTokens + kTaps - 1; ++j) x[j] = stacked_ld<T>(p.in, row + (size_t)j * p.in.row_stride);
+#pragma unroll
+    for (int i = 0; i < kPrepTokens; ++i) {
+      float acc = 0.0f;
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) acc += w[j] * x[i + j];
+      y[i] = acc / (1.0f + expf(-acc));
+    }
+  };
+  // kPrepTokens values of one channel, any run
+  auto channel = [&](int e, float (&y)[kPrepTokens]) {
+    float w[kTaps], win[kTaps];
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) { w[j] = p.taps[(size_t)(chan0 + e) * kTaps + j]; win[j] = 0.0f; }
+#pragma unroll
+    for (int i = 0; i < kPrepTokens; ++i) {
+      y[i] = 0.0f;
+      if (!ok[i]) continue;
+      const size_t row = (size_t)(t0 + i) * p.in.row_stride + col0 + e;
+      if (i == 0 || place[i] == 0 || !ok[i > 0 ? i - 1 : 0]) {        // the window starts anew
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j) {
+          const int s = place[i] - (kTaps - 1) + j;
+          win[j] = s >= 0 ? stacked_ld<T>(p.in, row - (size_t)(kTaps - 1 - j) * p.in.row_stride)
+                          : tails[i][(size_t)(kTaps - 1 + s) * channels + chan0 + e];
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j) win[j] = win[j + 1];
+      }
+      win[kTaps - 1] = stacked_ld<T>(p.in, row);
+      float acc = 0.0f;
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) acc += w[j] * win[j];
+      y[i] = acc / (1.0f + expf(-acc));
+    }
+  };
+  if (kind == 2) {
+#pragma unroll 2
+    for (int e = lane; e < d; e += 32) {
+      float y[kPrepTokens];
+      if (usual) usual_channel(e, y); else channel(e, y);
+#pragma unroll
+      for (int i = 0; i < kPrepTokens; ++i) {
+        if (ok[i]) dst[(size_t)i * dst_stride + e] = y[i];
+      }
+    }
+    if (p.channel_decay) {
+      const float rate = -expf(p.a_log[head]);
+#pragma unroll 2
+      for (int e = lane; e < p.dk; e += 32) {
+        const float bias = p.dt_bias[(size_t)head * p.dk + e];
+        float in[kPrepTokens];
+#pragma unroll
+        for (int i = 0; i < kPrepTokens; ++i) {
+          in[i] = i < cnt ? stacked_ld<T>(p.a_in, (size_t)(t0 + i) * p.a_in.row_stride + (size_t)head * p.dk + e) : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < kPrepTokens; ++i) {
+          if (!ok[i]) continue;
+          const float a = in[i] + bias;
+          const float sp = a > 20.0f ? a : log1pf(expf(a));
+          p.g_out[((size_t)(t0 + i) * p.heads + head) * p.dk + e] = expf(rate * sp);
+        }
+      }
+    }
+    if (lane < cnt) {
+      const int t = t0 + lane;
+      const size_t row = (size_t)t * p.in.row_stride;
+      const float b = stacked_ld<T>(p.in, row + p.b_off + head);
+      p.beta_out[(size_t)t * p.heads + head] = 1.0f / (1.0f + expf(-b));
+      if (!p.channel_decay) {
+        const float a = stacked_ld<T>(p.in, row + p.a_off + head) + p.dt_bias[head];
+        const float sp = a > 20.0f ? a : log1pf(expf(a));
+        p.g_out[(size_t)t * p.heads + head] = expf(-expf(p.a_log[head]) * sp);
+      }
+    }
+    return;
+  }
+  float y[8][kPrepTokens];            // key_dim <= 256
+#pragma unroll
+  for (int it = 0; it < 8; ++it) {
+#pragma unroll
+    for (int i = 0; i < kPrepTokens; ++i) y[it][i] = 0.0f;
+  }
+  if (usual) {
+#pragma unroll
+    for (int it = 0; it < 8; ++it) {
+      if (lane + 32 * it < d) usual_channel(lane + 32 * it, y[it]);
+    }
+  } else {
+#pragma unroll
+    for (int it = 0; it < 8; ++it) {
+      if (lane + 32 * it < d) channel(lane + 32 * it, y[it]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kPrepTokens; ++i) {
+    float ss = 0.0f;
+#pragma unroll
+    for (int it = 0; it < 8; ++it) {
+      if (32 * it < d) ss += warp_sum(y[it][i] * y[it][i]);
+    }
+    const float f = rsqrtf(ss + p.unit_eps) * (kind == 0 ? p.q_scale : 1.0f);
+#pragma unroll
+    for (int it = 0; it < 8; ++it) {
+      const int e = lane + 32 * it;
+      if (ok[i] && e < d) dst[(size_t)i * dst_stride + e] = y[it][i] * f;
+    }
+  }
+}
+
 // The record's tail after the step: the last K - 1 inputs of every channel.  One thread per
 // (request, channel) reads what it needs of the old tail before it writes.
 template <typename T>
@@ -504,12 +667,20 @@ TK_API int tk_delta_prepare(const void* x, const float* parts, int n_parts, long
   if (units > 65535 || dk > 256) return (int)cudaErrorInvalidValue;
   const int widest = dk > dv ? dk : dv;
   // few tokens: a block a unit, so that a step of single tokens is one memory latency long; many: a warp a unit
-  // (shape 1 / 2: the caller's choice, for tests and measurements; both give the same bits)
+  // (shape 1 / 2 / 3: a warp a unit, a block a unit, a warp a unit for several tokens in a row; the same bits)
   p.per_warp = shape == 1 ? 1 : shape == 2 ? 0 : ((long long)n_tokens * units >= 4096 ? 1 : 0);
   const int threads = p.per_warp ? tk::kDeltaPrepWarps * 32 : (widest >= 256 ? 256 : (widest + 31) / 32 * 32);
   dim3 grid(n_tokens, p.per_warp ? (units + tk::kDeltaPrepWarps - 1) / tk::kDeltaPrepWarps : units);
   cudaError_t e = cudaSuccess;
-  TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::delta_prepare_kernel<T>, grid, dim3(threads), 0, stream, p));
+  if ((shape == 3 || (shape == 0 && p.per_warp)) && !p.move_tail && n_taps >= 2 && n_taps <= 4) {
+    const dim3 rgrid((n_tokens + tk::kPrepTokens - 1) / tk::kPrepTokens, (units + tk::kDeltaPrepWarps - 1) / tk::kDeltaPrepWarps);
+#define TK_DELTA_ROWS(K) \
+    TK_DISPATCH_DTYPE(dtype, T, (e = tk::launch(tk::delta_prepare_rows_kernel<T, K>, rgrid, dim3(tk::kDeltaPrepWarps * 32), 0, stream, p)))
+    if (n_taps == 2) { TK_DELTA_ROWS(2); } else if (n_taps == 3) { TK_DELTA_ROWS(3); } else { TK_DELTA_ROWS(4); }
+#undef TK_DELTA_ROWS
+  } else {
+    TK_DISPATCH_DTYPE(dtype, T, e = tk::launch(tk::delta_prepare_kernel<T>, grid, dim3(threads), 0, stream, p));
+  }
   if (e != cudaSuccess || n_taps == 1 || p.move_tail) return (int)e;
   const int hk = kv_heads * dk, hv = heads * dv;
   dim3 tgrid((2 * hk + hv + 127) / 128, n_reqs);

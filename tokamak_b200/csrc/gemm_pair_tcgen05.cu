@@ -101,7 +101,6 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
   const int n_tiles = n_tm * n_tn;
   const int n_kb = (p.k + kGpBK - 1) / kGpBK;
 
-  pdl_trigger();
   if (threadIdx.x == 0) {
     for (int s = 0; s < kGpStages; ++s) {
       mbar_init(gt_smem_u32(&full_bar[s]), 1);
@@ -124,6 +123,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
   cluster_sync_all();            // both blocks' barriers exist before anything arrives on them
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
+  // only now may later kernels begin: none of them can take tensor memory before this block has its own
+  pdl_trigger();
 
   if (warp == 0) {
     // ---- TMA producer of this block's halves ---------------------------------------------------

@@ -1852,8 +1852,8 @@ def delta_prepare(proj: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, d
     (every request must bring at least one token: with as many tokens as requests the same kernel does both).
     ``channel_a`` (``[N, heads * key_dim]`` like ``proj``: type ``dtype`` or float32 partial sums): a decay per head and key
     channel from it instead of one per head; ``dt_bias`` is then ``[heads * key_dim]`` and ``g`` ``[N, H, dk]``.
-    ``shape``: 0 lets the launcher choose a warp (many tokens) or a block (few) per head, 1 and 2 force one;
-    the results are the same bits.
+    ``shape``: 0 lets the launcher choose by the number of tokens; 1 (a warp per head), 2 (a block per head) and 3 (a warp
+    per head for several tokens in a row; 2 to 4 taps) force one; the results are the same bits.
     Returns ``(q [N, Hk, dk], k [N, Hk, dk], v [N, H, dv], beta [N, H], g [N, H])``."""
     _want(taps, torch.float32, "taps"); _want(a_log, torch.float32, "a_log"); _want(dt_bias, torch.float32, "dt_bias")
     _want(records, torch.float32, "records")

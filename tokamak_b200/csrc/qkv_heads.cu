@@ -308,22 +308,24 @@ __global__ void qkv_heads_vec_kernel(QkvHeadsParams p) {
 
 // The same for pieces of up to 128 elements (sizes, offsets and row lengths multiples of 4, the rotated part in whole
 // fours per half, values of their own): kLanes lanes take a piece, four elements each, so that a warp works on 32 /
-// kLanes pieces, and rotation partners and sums of squares pass between lanes instead of through shared memory.
+// kLanes pieces (a value head longer than that is cut: nothing passes between its elements), and rotation partners and sums of squares pass between lanes instead of through shared memory.
 template <typename T, int kLanes>
 __global__ void __launch_bounds__(kHeadsWarps * 32) qkv_heads_lanes_kernel(QkvHeadsParams p) {
   constexpr int kPieces = 32 / kLanes;
   pdl_trigger();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int first = (blockIdx.y * kHeadsWarps + warp) * kPieces;
-  const int k_heads = p.n_kv_heads * p.maps, heads_total = p.n_q_heads + k_heads + p.n_kv_heads;
+  const int v_cuts = (p.v_dim + 4 * kLanes - 1) / (4 * kLanes);
+  const int k_heads = p.n_kv_heads * p.maps, heads_total = p.n_q_heads + k_heads + p.n_kv_heads * v_cuts;
   if (first >= heads_total) return;                    // the whole warp
   const int t = blockIdx.x;
   const int h = min(first + lane / kLanes, heads_total - 1);
   const bool real = first + lane / kLanes < heads_total;
   const int kind = h < p.n_q_heads ? 0 : h < p.n_q_heads + k_heads ? 1 : 2;       // 0 = q, 1 = k, 2 = v
-  const int head = kind == 0 ? h : kind == 1 ? h - p.n_q_heads : h - p.n_q_heads - k_heads;
+  const int v_item = h - p.n_q_heads - k_heads;
+  const int head = kind == 0 ? h : kind == 1 ? h - p.n_q_heads : v_item / v_cuts;
   const int d = kind == 2 ? p.v_dim : p.k_dim;
-  const int c = lane % kLanes, e = 4 * c;
+  const int c = lane % kLanes, e = 4 * (c + (kind == 2 ? (v_item % v_cuts) * kLanes : 0));
   const bool live = real && e < d;
   const int r = p.rope_table != nullptr && kind != 2 ? p.rotary_dim : 0, half = r >> 1;
   pdl_wait();
@@ -423,9 +425,10 @@ __global__ void __launch_bounds__(kHeadsWarps * 32) qkv_heads_lanes_kernel(QkvHe
     }
     return;
   }
-  for (int i = d + e; i < tail; i += 4 * kLanes) st4<T>(dst + off + i, zero4);
+  const int step = 4 * kLanes * (kind == 2 ? v_cuts : 1);
+  for (int i = d + e; i < tail; i += step) st4<T>(dst + off + i, zero4);
   for (int z = 1; z <= zero_rows; ++z) {
-    for (int i = e; i < tail; i += 4 * kLanes) st4<T>(dst + (size_t)z * row_len + off + i, zero4);
+    for (int i = e; i < tail; i += step) st4<T>(dst + (size_t)z * row_len + off + i, zero4);
   }
 }
 
@@ -467,11 +470,11 @@ TK_API int tk_qkv_heads(const void* x, const float* parts, int n_parts, long lon
   cudaError_t e = cudaSuccess;
   const bool vec = k_dim % 4 == 0 && v_dim % 4 == 0 && k_row % 4 == 0 && v_row % 4 == 0 && row_stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
                    (v_off < 0 || v_off % 4 == 0);
-  const int widest = k_dim > v_dim ? k_dim : v_dim;
-  if (vec && widest <= 128 && v_off >= 0 && (rope_table == nullptr || rotary_dim % (halves ? 8 : 4) == 0) &&
+  if (vec && k_dim <= 128 && v_off >= 0 && (rope_table == nullptr || rotary_dim % (halves ? 8 : 4) == 0) &&
       ((uintptr_t)rope_table & 15) == 0) {
-    const int lanes = widest <= 32 ? 8 : widest <= 64 ? 16 : 32, per_block = tk::kHeadsWarps * (32 / lanes);
-    const dim3 g((unsigned)n_tokens, (unsigned)((heads_total + per_block - 1) / per_block));
+    const int lanes = k_dim <= 32 ? 8 : k_dim <= 64 ? 16 : 32, per_block = tk::kHeadsWarps * (32 / lanes);
+    const int items = n_q_heads + n_kv_heads * maps + n_kv_heads * ((v_dim + 4 * lanes - 1) / (4 * lanes));
+    const dim3 g((unsigned)n_tokens, (unsigned)((items + per_block - 1) / per_block));
 #define TK_QKV_LANES(L) \
     TK_DISPATCH_DTYPE(dtype, T, (e = tk::launch(tk::qkv_heads_lanes_kernel<T, L>, g, dim3(tk::kHeadsWarps * 32), 0, stream, p)))
     if (lanes == 8) { TK_QKV_LANES(8); } else if (lanes == 16) { TK_QKV_LANES(16); } else { TK_QKV_LANES(32); }
