@@ -210,10 +210,10 @@ class DecoderModel:
             pending = self._join(resid, pending, call.joins, embedded, getattr(block, "entry_norm", None))
             if getattr(block, "TAKES_NEXT_NORM", False):
                 # the norm that will consume what the block leaves pending: the next block's, or the last; none
-                # where more joins the stream before it
+                # where more joins the stream before it or the reader behind it cannot pay an owed scale
                 after = self.blocks[schedule[i + 1].block] if i + 1 < len(schedule) else None
                 next_norm = getattr(after, "entry_norm", None) if after is not None else self.final_norm
-                if after is not None and schedule[i + 1].joins is not None:
+                if after is not None and (schedule[i + 1].joins is not None or not getattr(after, "entry_takes_owed", True)):
                     next_norm = None
                 resid, pending = block.forward(resid, pending, step, view, next_norm=next_norm)
             else:

@@ -60,7 +60,8 @@ feed-forward with ``TAKES_THEN_NORM = True`` is called with ``then_norm=(resid, 
 may return an :class:`OwedNorm` prepared for that norm instead of its output; one with
 ``TAKES_OWED_NORM = True`` may be handed an :class:`OwedNorm` as ``h`` (others get a tensor); a
 block with ``TAKES_NEXT_NORM = True`` is told which norm will consume what it leaves pending and
-names the norm that consumes its own input as ``entry_norm``.  Parts without these attributes
+names the norm that consumes its own input as ``entry_norm`` (``entry_takes_owed = False``: the part behind it does not
+take an :class:`OwedNorm`, and nobody prepares one for it).  Parts without these attributes
 never see any of it.
 
 **Queued products.**  In those same steps the products of consecutive parts (attention output,

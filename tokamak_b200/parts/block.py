@@ -92,6 +92,10 @@ class PreNormBlock:
     def entry_norm(self):
         return self.norm1
 
+    @property
+    def entry_takes_owed(self) -> bool:
+        return getattr(self.mixer, "TAKES_OWED_NORM", False)
+
     @staticmethod
     def _branch(part, h, args: tuple, then_norm):
         if isinstance(h, OwedNorm) and not getattr(part, "TAKES_OWED_NORM", False):
@@ -105,7 +109,9 @@ class PreNormBlock:
         then = (resid, next_norm) if next_norm is not None else None
         if self.feed_forward is None:
             return resid, self._branch(self.mixer, h, (step, cache_view), then)
-        a = self._branch(self.mixer, h, (step, cache_view), (resid, self.norm2))
+        # a mixer prepares the next norm's input only for a feed-forward that can pay the owed scale itself
+        owed = getattr(self.feed_forward, "TAKES_OWED_NORM", False)
+        a = self._branch(self.mixer, h, (step, cache_view), (resid, self.norm2) if owed else None)
         h = self.norm2.add_norm(resid, a)
         if getattr(self.feed_forward, "LEAVES_WEIGHTED_ROWS", False):
             return resid, SumBranch(self._terms(self.feed_forward, h, step))
