@@ -1784,14 +1784,14 @@ def puresun_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
 # attention beside a recurrent half in one layer and mixtures with groups of experts); its delta rule's kernels
 # beside Logivik's, its attention's beside those of Ketalix
 
-SOFINEX_EXPERTS, SOFINEX_IDENTITY, SOFINEX_TOP, SOFINEX_RANK = 12, 4, 4, 128
+SOFINEX_EXPERTS, SOFINEX_IDENTITY, SOFINEX_TOP, SOFINEX_RANK = 22, 2, 3, 128
 
 
 def sofinex_config(s: dict) -> dict:
     """Parallel layers (windowed attention with sinks beside the delta rule: width / 128 heads of 128 x 128, low-rank
     projections of 128) with an ungated feed-forward that holds as many weights as a gated one of width ff, and
-    differential attention layers (two maps of half a head's size over the twin's value heads) with a mixture: 12
-    experts and 4 identity experts of which 4 are used, a shared expert, ff / 4 each.  Two of the layers run twice, so
+    differential attention layers (two maps of half a head's size over the twin's value heads) with a mixture: 22
+    experts and 2 identity experts of which 3 are used, a shared expert, ff / 4 each.  Two of the layers run twice, so
     that there are as many layer runs as the twin has layers."""
     w, d = s["width"], s["dim"]
     att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "vdim": d, "mask": {"size": s["window"]}}
@@ -1802,7 +1802,7 @@ def sofinex_config(s: dict) -> dict:
     right = {"heads": w // 128, "kv_heads": w // 128, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": SOFINEX_RANK,
              "gate_rank": SOFINEX_RANK}
     moe = {"kind": "moe", "expert": {"ff": s["ff"] // 4}, "shared": {"ff": s["ff"] // 4},
-           "router": {"experts": SOFINEX_EXPERTS, "identity": SOFINEX_IDENTITY, "top": SOFINEX_TOP, "groups": {"count": 4, "keep": 3}}}
+           "router": {"experts": SOFINEX_EXPERTS, "identity": SOFINEX_IDENTITY, "top": SOFINEX_TOP, "groups": {"count": 6, "keep": 4}}}
     layers = [{"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": {"kind": "dense", "ff": s["ff"] * 3 // 2}}
               if i % 2 == 0 else {"type": "attention", "mixer": diff, "mlp": moe} for i in range(s["layers"] - 2)]
     return {"architecture": "Sofinex", "vocab": s["vocab"], "width": w, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
@@ -1964,14 +1964,14 @@ def sofinex_kernels(s: dict, tokens: int, batch: int, ctx: int, peaks: dict) -> 
         row(f"up product with the exact gelu, {name}", f"up product with relu squared, {name}", t_us(up("gelu")), t_us(up("relu2")),
             **(dict(nbytes=w_up.numel() * 2) if single else dict(flops=2.0 * n * ff * width)))
         # ---- the experts
-        rk = dict(top=top, n_groups=4, keep=3, padded=True)
+        rk = dict(top=top, n_groups=6, keep=4, padded=True)
         mine = lambda: ops.moe_route(h, router, corr, kind="softmax_all", group_score="best", normalize=True, identity=identity,
                                      shared=1, **rk)
         row(f"router over all outputs, identity and shared experts, {name}", f"sigmoid router with groups, {name}",
             t_us(mine), t_us(lambda: ops.moe_route(h, router[:-1], corr, **rk)),
             nbytes=n * width * 2 + router.numel() * 4)
         routing = mine()
-        plain_r = ops.moe_route(h, router[:experts].contiguous(), None, **rk)
+        plain_r = ops.moe_route(h, router[:experts].contiguous(), None, top=top, padded=True)
         small = ops.moe_small_takes(n, top + 1, width, ffe)
         run = lambda r, wa, wb, small: ((lambda: ops.moe_experts_small(h, r, wa, wb, combine=False)) if small else
                                         (lambda: ops.moe_experts_tc(h, r, wa, wb, err, combine=False)))

@@ -86,9 +86,9 @@ SX_D = {
     "loop": {"start": 1, "stop": 3, "times": 1},
     "layers": [
         _diff_layer(_att(2, 1, 64, 128, 0.1, 20, 32, 10000.0, _wave(2.0, 1.0, 4.0, 100)), 0.5, _dense(384)),
-        _pair_layer(_att(4, 1, 128, 96, 0.06, 100, 128, 250000.0, _yarn(4.0, 256, 32.0, 1.0)), _delta(3, 3, 64, 48, 2, 40, 72),
+        _pair_layer(_att(4, 1, 128, 96, 0.06, 100, 128, 150000.0, _yarn(4.0, 256, 32.0, 1.0)), _delta(3, 3, 64, 48, 2, 40, 72),
                     _moe(128, 10, 6, 5, 4, 2, 200)),
-        _pair_layer(_att(2, 2, 70, 130, 0.1, 16, 60, 3000.0, None), _delta(2, 1, 136, 24, 5, 24, 24), _dense(100)),
+        _pair_layer(_att(2, 2, 70, 130, 0.1, 16, 60, 3000.0, None), _delta(2, 1, 136, 24, 5, 26, 18), _dense(100)),
     ],
 }
 # (configuration, how the random weights are drawn, page size)

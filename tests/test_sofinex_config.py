@@ -143,7 +143,7 @@ def test_frequencies_stretched_by_wavelength(dims, base, factor, low, high, orig
 
 
 @pytest.mark.parametrize("dims,base,factor,original,fast,slow", [
-    (96, 10000.0, 4.0, 512, 32.0, 1.0), (8, 500.0, 2.0, 64, 8.0, 2.0), (4, 100.0, 16.0, 4096, 32.0, 1.0), (64, 1e6, 1.0, 100, 4.0, 4.0)])
+    (80, 10000.0, 5.0, 600, 24.0, 1.0), (8, 500.0, 2.0, 64, 8.0, 2.0), (4, 100.0, 16.0, 4096, 32.0, 1.0), (64, 1e6, 1.0, 100, 4.0, 4.0)])
 def test_frequencies_stretched_by_pair_index(dims, base, factor, original, fast, slow):
     got, mag = scaled_frequencies(dims, base, YarnScaling(factor, original, fast, slow))
     want, wmag = plain.ramped_frequencies(dims, base, {"factor": factor, "original": original, "fast": fast, "slow": slow})
